@@ -1,15 +1,18 @@
 from .errors import ConfigError, UnknownArchitectureError
 from .reader import KeyReader, read_config_json
-from .spec import LayerSpec, ModelSpec, PartSpec
+from .spec import LayerSpec, ModelSpec, PartSpec, PassStart
 from .mistral import MistralConfig
 from .kikopel import KikopelConfig
 from .tovapel import TovapelConfig
 from .rupasun import RupasunConfig
+from .fezolorn import FezolornConfig
+from .dunesun import DunesunConfig
 from .registry import (architecture_names, config_from_dict, load_config,
                        register_architecture)
 
 __all__ = [
     "ConfigError", "UnknownArchitectureError", "KeyReader", "read_config_json",
-    "LayerSpec", "ModelSpec", "PartSpec", "MistralConfig", "KikopelConfig", "TovapelConfig", "RupasunConfig", "architecture_names",
+    "LayerSpec", "ModelSpec", "PartSpec", "PassStart", "MistralConfig", "KikopelConfig", "TovapelConfig", "RupasunConfig",
+    "FezolornConfig", "DunesunConfig", "architecture_names",
     "config_from_dict", "load_config", "register_architecture",
 ]

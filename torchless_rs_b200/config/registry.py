@@ -67,6 +67,8 @@ def _register_builtin() -> None:
     register_architecture("Rupasun")(RupasunConfig)
     from .fezolorn import FezolornConfig
     register_architecture("Fezolorn")(FezolornConfig)
+    from .dunesun import DunesunConfig
+    register_architecture("Dunesun")(DunesunConfig)
 
 
 _register_builtin()

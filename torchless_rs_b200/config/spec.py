@@ -54,6 +54,15 @@ class LayerSpec:
 
 
 @dataclass(frozen=True)
+class PassStart:
+    """What is added to the stream right before an entry of the order runs (the first layer of a pass through
+    layers that run several times): a row of the model's `pass_table_name`, and, if asked for, the embedded
+    tokens (the stream as it was before the first layer)."""
+    row: Optional[int] = None
+    add_embedded: bool = False
+
+
+@dataclass(frozen=True)
 class ModelSpec:
     """A whole decoder.  `order` lists indices into `layers` in the order in which
     they run; an index may appear more than once."""
@@ -78,6 +87,9 @@ class ModelSpec:
     streams: Optional[int] = None                # residual streams kept side by side: every one starts as
                                                  #   the embedded token, the layers' blocks read and write
                                                  #   all of them, their sum goes to the final norm
+    pass_starts: Mapping[int, PassStart] = field(default_factory=dict)   # place in `order` -> what is added there
+    pass_table_name: Optional[str] = None        # a table [pass_rows, hidden] for the passes' rows
+    pass_rows: int = 0
 
     def validate(self) -> None:
         from .errors import ConfigError
@@ -97,6 +109,13 @@ class ModelSpec:
         for i in self.order:
             if not 0 <= i < n:
                 raise ConfigError(f"layer order names layer {i}, but there are {n} layers")
+        for k, start in self.pass_starts.items():
+            if not 0 <= k < len(self.order):
+                raise ConfigError(f"something is added before entry {k} of the order, which has {len(self.order)}")
+            if start.row is not None and (self.pass_table_name is None or not 0 <= start.row < self.pass_rows):
+                raise ConfigError(f"entry {k} of the order adds row {start.row} of a table of {self.pass_rows} rows")
+        if self.pass_starts and self.streams is not None:
+            raise ConfigError("a model with several residual streams adds nothing between its layers")
         first_run = {}
         for step, i in enumerate(self.order):
             first_run.setdefault(i, step)

@@ -11,7 +11,8 @@
 // table and the first layer are taken here, since this kernel writes the stream anyway:
 // a multiplier (`scale`, 1 = none) and a learned row per position (`pos_table`
 // [max_pos, H] with `token_pos`, null = none): x[t, :] = scale * table[tok, :] +
-// pos_table[token_pos[t], :], in 32-bit.
+// pos_table[token_pos[t], :], in 32-bit.  `copy` (null = none) keeps the embedded tokens for layers that add
+// them again later; `add_vec` (null = none) is then added to the stream alone.
 // ---------------------------------------------------------------------------
 // A token may also be taken from a device buffer (the tokens that the previous step selected):
 // with `token_src` given, token t is token_src[token_from[t]] wherever token_from[t] >= 0.
@@ -19,7 +20,7 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restri
                              const int* __restrict__ token_src, const act_t* __restrict__ table,
                              float* __restrict__ x, int H, int vocab, float scale,
                              const act_t* __restrict__ pos_table, const int* __restrict__ token_pos,
-                             int max_pos) {
+                             int max_pos, float* __restrict__ copy, const float* __restrict__ add_vec) {
   TL_TRACE_SCOPE(1, H, 1);
   pdl_wait();
   TL_TRACE_RELEASED();
@@ -30,7 +31,19 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restri
   tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);  // the host has checked the range already
   const act_t* src = table + (size_t)tok * H;
   float* dst = x + (size_t)t * H;
-  if (pos_table == nullptr) {
+  if (copy != nullptr || add_vec != nullptr) {
+    const act_t* pr = nullptr;
+    if (pos_table != nullptr) {
+      int p = token_pos[t];
+      p = p < 0 ? 0 : (p >= max_pos ? max_pos - 1 : p);
+      pr = pos_table + (size_t)p * H;
+    }
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float v = pr != nullptr ? fmaf(scale, to_f32(src[i]), to_f32(pr[i])) : scale * to_f32(src[i]);
+      if (copy != nullptr) copy[(size_t)t * H + i] = v;
+      dst[i] = add_vec != nullptr ? v + add_vec[i] : v;
+    }
+  } else if (pos_table == nullptr) {
     for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = scale * to_f32(src[i]);
   } else {
     int p = token_pos[t];
@@ -42,12 +55,13 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restri
 
 extern "C" int TL_NAME(tl_embed)(const int* tokens, const int* token_from, const int* token_src,
                                  const void* table, float* x, int T, int H, int vocab, float scale,
-                                 const void* pos_table, const int* token_pos, int max_pos,
-                                 cudaStream_t stream) {
+                                 const void* pos_table, const int* token_pos, int max_pos, float* copy,
+                                 const float* add_vec, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (pos_table != nullptr && (token_pos == nullptr || max_pos <= 0)) return TL_ERR_BAD_ARG;
   return tl_launch(embed_kernel, dim3(T), dim3(256), 0, stream, tokens, token_from, token_src,
-                   (const act_t*)table, x, H, vocab, scale, (const act_t*)pos_table, token_pos, max_pos);
+                   (const act_t*)table, x, H, vocab, scale, (const act_t*)pos_table, token_pos, max_pos,
+                   copy, add_vec);
 }
 
 // ---------------------------------------------------------------------------

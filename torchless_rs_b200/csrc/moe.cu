@@ -5,7 +5,7 @@
 //   the `top` largest (ties: the lower index); the weights are the chosen s, not renormalised.
 //   Router outputs from `experts` on have no matrices: such an expert hands its input through.
 //   A real expert: g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit),
-//                  y = W_down( g * sigmoid(alpha g) * (u + 1) ).
+//                  y = W_down( g * sigmoid(alpha g) * (u + 1) ), or the plain y = W_down( silu(W_gate h) (W_up h) ).
 //
 // Nothing here needs the host: counts and offsets stay on the device, and the product kernels are
 // launched over an upper bound of tiles, of which a block finds its own (expert, rows) or leaves.
@@ -176,6 +176,67 @@ extern "C" int TL_NAME(tl_moe_route_grouped)(const float* z, int ldz, int n_out,
                    dim3(MOE_GROUPED_WARPS * 32), 0, stream, z, ldz, n_out, groups, keep, top, scale, idx, wt, T);
 }
 
+// The choice by the logits themselves: l = z + bias (32-bit); the `top` largest l are chosen (ties: the lower
+// index), their weights are the softmax over the chosen l alone.  A warp per token.
+__global__ void __launch_bounds__(256)
+moe_route_chosen_kernel(const float* __restrict__ z, int ldz, const float* __restrict__ bias, int n_out, int top,
+                        int* __restrict__ idx, float* __restrict__ wt, int T) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31;
+  const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (t >= T) return;
+  const float* row = z + (size_t)t * ldz;
+  float l[MOE_MAX_PER_LANE];
+#pragma unroll
+  for (int r = 0; r < MOE_MAX_PER_LANE; ++r) {
+    const int e = lane + 32 * r;
+    l[r] = e < n_out ? row[e] + (bias != nullptr ? bias[e] : 0.0f) : -INFINITY;
+  }
+  unsigned taken = 0;                          // bit r: this lane's output 32 r + lane is chosen already
+  float first = 0.0f, sum = 0.0f;              // the largest logit; the sum of exp(l - largest)
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int best_e = 0x7fffffff;
+#pragma unroll
+    for (int r = 0; r < MOE_MAX_PER_LANE; ++r) {
+      const int e = lane + 32 * r;
+      if (e < n_out && !(taken >> r & 1) && (l[r] > best || best_e == 0x7fffffff)) {   // a tie keeps the lower index
+        best = l[r];
+        best_e = e;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+      if (oe != 0x7fffffff && (best_e == 0x7fffffff || ob > best || (ob == best && oe < best_e))) {
+        best = ob;
+        best_e = oe;
+      }
+    }
+    if (k == 0) first = best;
+    const float w = expf(best - first);
+    sum += w;
+    if (lane == 0) {
+      idx[(size_t)t * top + k] = best_e;
+      wt[(size_t)t * top + k] = w;
+    }
+    if ((best_e & 31) == lane) taken |= 1u << (best_e >> 5);
+  }
+  __syncwarp();
+  for (int k = lane; k < top; k += 32) wt[(size_t)t * top + k] /= sum;
+}
+
+extern "C" int TL_NAME(tl_moe_route_chosen)(const float* z, int ldz, const float* bias, int n_out, int top, int* idx,
+                                            float* wt, int T, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (n_out < 1 || top < 1 || top > n_out) return TL_ERR_BAD_ARG;
+  if (n_out > 32 * MOE_MAX_PER_LANE) return TL_ERR_UNSUPPORTED;
+  return tl_launch(moe_route_chosen_kernel, dim3((T + 7) / 8), dim3(256), 0, stream, z, ldz, bias, n_out, top, idx,
+                   wt, T);
+}
+
 // Groups the pairs by expert.  offsets[e] .. offsets[e + 1] are the rows of expert e < E in the
 // grouped order; row_token[row] is the token a row belongs to; row_of[pair] is the row of pair
 // (t, k), or -1 for a pair whose expert hands its input through.  One block: the pairs of a step
@@ -241,11 +302,22 @@ extern "C" int TL_NAME(tl_moe_plan)(const int* idx, int n_pairs, int top, int E,
 #define GBN 64
 #define GBK 16
 
+// What the gate and up sums of an expert go through: kind 0 silu(g) u; kind 2 the clamped form
+// g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1).
+#define MOE_ACT_SILU 0
+#define MOE_ACT_CLAMPED 2
+__device__ __forceinline__ float moe_act(float g, float u, int kind, float limit, float alpha) {
+  if (kind == MOE_ACT_SILU) return g / (1.0f + expf(-g)) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+
 template <bool UP>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const act_t* __restrict__ A, int lda, const int* __restrict__ row_token,
                 const act_t* __restrict__ W, void* __restrict__ C, int ldc, const int* __restrict__ offsets,
-                int E, int N, int K, float limit, float alpha) {
+                int E, int N, int K, int kind, float limit, float alpha) {
   __shared__ float As[GBK][GBM + 4];
   __shared__ float Ws[GBK][GBN + 4];
   __shared__ float Us[UP ? GBK : 1][GBN + 4];
@@ -324,9 +396,7 @@ moe_gemm_kernel(const act_t* __restrict__ A, int lda, const int* __restrict__ ro
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       if (UP) {
-        const float g = fminf(acc[i][j], limit);
-        const float u = fminf(fmaxf(acu[i][j], -limit), limit);
-        ((act_t*)C)[(size_t)(r0 + m) * ldc + n] = from_f32<act_t>(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
+        ((act_t*)C)[(size_t)(r0 + m) * ldc + n] = from_f32<act_t>(moe_act(acc[i][j], acu[i][j], kind, limit, alpha));
       } else {
         ((float*)C)[(size_t)(r0 + m) * ldc + n] = acc[i][j];
       }
@@ -335,7 +405,7 @@ moe_gemm_kernel(const act_t* __restrict__ A, int lda, const int* __restrict__ ro
 }
 
 extern "C" int TL_NAME(tl_moe_gemm)(const void* A, int lda, const int* row_token, const void* W, void* C, int ldc,
-                                    const int* offsets, int E, int max_rows, int N, int K, int up, float limit,
+                                    const int* offsets, int E, int max_rows, int N, int K, int up, int kind, float limit,
                                     float alpha, cudaStream_t stream) {
   if (max_rows <= 0 || E <= 0) return 0;
   if (N < 1 || K < 1) return TL_ERR_BAD_ARG;
@@ -344,9 +414,9 @@ extern "C" int TL_NAME(tl_moe_gemm)(const void* A, int lda, const int* row_token
   dim3 grid((N + GBN - 1) / GBN, tiles);
   if (up)
     return tl_launch(moe_gemm_kernel<true>, grid, dim3(256), 0, stream, (const act_t*)A, lda, row_token,
-                     (const act_t*)W, C, ldc, offsets, E, N, K, limit, alpha);
+                     (const act_t*)W, C, ldc, offsets, E, N, K, kind, limit, alpha);
   return tl_launch(moe_gemm_kernel<false>, grid, dim3(256), 0, stream, (const act_t*)A, lda, row_token,
-                   (const act_t*)W, C, ldc, offsets, E, N, K, limit, alpha);
+                   (const act_t*)W, C, ldc, offsets, E, N, K, kind, limit, alpha);
 }
 
 // out[t, :] (+)= sum_k wt[t, k] * ( row_of[t, k] >= 0 ? yk[row_of[t, k], :] : h[t, :] ), k in order.
@@ -436,7 +506,7 @@ template <bool UP>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ row_token,
                     const bf16* __restrict__ W, void* __restrict__ C, int ldc, const int* __restrict__ offsets,
-                    int E, int N, int K, float limit, float alpha) {
+                    int E, int N, int K, int kind, float limit, float alpha) {
   __shared__ __align__(128) bf16 As[MSTAGES][MBM * MBK];
   __shared__ __align__(128) bf16 Ws[MSTAGES][MBN * MBK];
   __shared__ __align__(128) bf16 Us[UP ? MSTAGES : 1][UP ? MBN * MBK : 8];
@@ -544,9 +614,8 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__
         if (c + j >= N) continue;
         const float v = acc[n][half * 2 + j];
         if (UP) {
-          const float g = fminf(v, limit);
-          const float u = fminf(fmaxf(acu[n][half * 2 + j], -limit), limit);
-          ((bf16*)C)[(size_t)(r0 + m) * ldc + c + j] = __float2bfloat16_rn(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
+          ((bf16*)C)[(size_t)(r0 + m) * ldc + c + j] =
+              __float2bfloat16_rn(moe_act(v, acu[n][half * 2 + j], kind, limit, alpha));
         } else {
           ((float*)C)[(size_t)(r0 + m) * ldc + c + j] = v;
         }
@@ -556,7 +625,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__
 }
 
 extern "C" int tl_moe_gemm_mma(const void* A, int lda, const int* row_token, const void* W, void* C, int ldc,
-                               const int* offsets, int E, int max_rows, int N, int K, int up, float limit,
+                               const int* offsets, int E, int max_rows, int N, int K, int up, int kind, float limit,
                                float alpha, cudaStream_t stream) {
   if (max_rows <= 0 || E <= 0) return 0;
   if (N < 1 || K < 1) return TL_ERR_BAD_ARG;
@@ -566,8 +635,8 @@ extern "C" int tl_moe_gemm_mma(const void* A, int lda, const int* row_token, con
   dim3 grid((N + MBN - 1) / MBN, tiles);
   if (up)
     return tl_launch(moe_gemm_mma_kernel<true>, grid, dim3(128), 0, stream, (const bf16*)A, lda, row_token,
-                     (const bf16*)W, C, ldc, offsets, E, N, K, limit, alpha);
+                     (const bf16*)W, C, ldc, offsets, E, N, K, kind, limit, alpha);
   return tl_launch(moe_gemm_mma_kernel<false>, grid, dim3(128), 0, stream, (const bf16*)A, lda, row_token,
-                   (const bf16*)W, C, ldc, offsets, E, N, K, limit, alpha);
+                   (const bf16*)W, C, ldc, offsets, E, N, K, kind, limit, alpha);
 }
 #endif

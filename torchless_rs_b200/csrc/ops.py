@@ -141,7 +141,8 @@ class CoreOps:
                      "tl_moe_route", "tl_moe_plan", "tl_moe_gemm", "tl_moe_combine", "tl_moe_route_grouped",
                      "tl_rotary_cache_write", "tl_diff_heads", "tl_sigmoid_gate", "tl_norm_add_norm", "tl_relu_squared",
                      "tl_clamped_glu", "tl_delta_prep", "tl_conv_state_update", "tl_delta_scan", "tl_silu_rows",
-                     "tl_weighted_sum"):
+                     "tl_weighted_sum", "tl_close_block", "tl_moe_route_chosen", "tl_qk_whole_norm_cache_write",
+                     "tl_ssd_prep", "tl_ssd_walk", "tl_ssd_gate_norm"):
             fn = getattr(self.lib, f"{base}_{self.suffix}")
             fn.restype = c_int
             setattr(self, "_" + base, fn)
@@ -151,10 +152,12 @@ class CoreOps:
               token_from: Optional[torch.Tensor] = None,
               token_src: Optional[torch.Tensor] = None, scale: float = 1.0,
               position_table: Optional[torch.Tensor] = None,
-              token_pos: Optional[torch.Tensor] = None) -> None:
+              token_pos: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None,
+              add_vec: Optional[torch.Tensor] = None) -> None:
         """x[t] = scale * table[token t] (+ position_table[token_pos[t]]).  With `token_src`
         (int32 on the device), token t is token_src[token_from[t]] wherever token_from[t] >= 0,
-        else tokens[t]."""
+        else tokens[t].  `copy` (32-bit, the stream's shape) receives the same; `add_vec` (32-bit, one number
+        per coordinate) is then added to x alone."""
         _need(tokens, torch.int32, "embed tokens")
         _need(table, self.act_dtype, "embed table")
         _need(x, torch.float32, "embed out")
@@ -169,11 +172,17 @@ class CoreOps:
             if position_table.shape[1] != H:
                 raise KernelError("embed: the position table's width is not the stream's")
             max_pos = position_table.shape[0]
+        if copy is not None:
+            _need(copy, torch.float32, "embed copy")
+        if add_vec is not None:
+            _need(add_vec, torch.float32, "embed addend")
+        if (copy is not None and copy.shape != x.shape) or (add_vec is not None and add_vec.numel() != H):
+            raise KernelError("embed: the copy or the addend does not have the stream's size")
         _check(self._tl_embed(_ptr(tokens), _ptr(token_from if token_src is not None else None),
                               _ptr(token_src), _ptr(table), _ptr(x), c_int(T), c_int(H),
                               c_int(table.shape[0]), c_float(scale), _ptr(position_table),
                               _ptr(token_pos if position_table is not None else None), c_int(max_pos),
-                              _stream()), "embed")
+                              _ptr(copy), _ptr(add_vec), _stream()), "embed")
 
     def convert_into(self, src: torch.Tensor, dst: torch.Tensor) -> None:
         """dst (activation type, contiguous, on the device) = src (32-bit, bfloat16 or float16, the
@@ -924,6 +933,22 @@ class CoreOps:
                                           c_int(top), c_float(scale), _ptr(idx), _ptr(wt), c_int(T), _stream()),
                "moe_route_grouped")
 
+    def moe_route_chosen(self, z: torch.Tensor, bias: Optional[torch.Tensor], top: int, idx: torch.Tensor,
+                         wt: torch.Tensor) -> None:
+        """idx[t, :top] = the largest z[t] + bias (ties: the lower index), wt = the softmax over those alone."""
+        _need(z, torch.float32, "router logits", contiguous=False)
+        _need(idx, torch.int32, "chosen experts")
+        _need(wt, torch.float32, "expert weights")
+        T, n_out = z.shape
+        if z.stride(1) != 1 or idx.shape != (T, top) or wt.shape != (T, top):
+            raise KernelError("moe_route_chosen: sizes do not match")
+        if bias is not None:
+            _need(bias, torch.float32, "router bias")
+            if bias.numel() != n_out:
+                raise KernelError("moe_route_chosen: the bias has one entry per expert")
+        _check(self._tl_moe_route_chosen(_ptr(z), c_int(z.stride(0)), _ptr(bias), c_int(n_out), c_int(top), _ptr(idx),
+                                         _ptr(wt), c_int(T), _stream()), "moe_route_chosen")
+
     def moe_plan(self, idx: torch.Tensor, experts: int, offsets: torch.Tensor, row_token: torch.Tensor,
                  row_of: torch.Tensor) -> None:
         """Groups the (token, choice) pairs by expert: offsets [experts + 1], row_token [pairs], row_of
@@ -937,9 +962,13 @@ class CoreOps:
                                  _ptr(row_token), _ptr(row_of), _stream()), "moe_plan")
 
     def moe_gemm(self, a: torch.Tensor, row_token: Optional[torch.Tensor], w: torch.Tensor, c: torch.Tensor,
-                 offsets: torch.Tensor, up: bool, limit: float = 0.0, alpha: float = 0.0) -> None:
+                 offsets: torch.Tensor, up: bool, limit: float = 0.0, alpha: float = 0.0,
+                 act: int = ACT_CLAMPED_GLU) -> None:
         """The experts' products over rows grouped by expert.  up: c[row] = act(gate, up) of a[row_token[row]]
-        with w [experts, 2 N, K]; else c[row] (32-bit) = a[row] . w[expert] with w [experts, N, K]."""
+        with w [experts, 2 N, K] (`act`: ACT_CLAMPED_GLU with `limit` and `alpha`, or ACT_PLAIN, silu(gate) * up);
+        else c[row] (32-bit) = a[row] . w[expert] with w [experts, N, K]."""
+        if act not in (ACT_PLAIN, ACT_CLAMPED_GLU):
+            raise KernelError(f"moe_gemm: no such activation ({act})")
         _need(a, self.act_dtype, "expert input")
         _need(w, self.act_dtype, "expert matrices")
         _need(c, self.act_dtype if up else torch.float32, "expert output")
@@ -952,12 +981,13 @@ class CoreOps:
             self.lib.tl_moe_gemm_mma.restype = c_int
             st = self.lib.tl_moe_gemm_mma(_ptr(a), c_int(a.stride(0)), _ptr(row_token), _ptr(w), _ptr(c),
                                           c_int(c.stride(0)), _ptr(offsets), c_int(E), c_int(c.shape[0]), c_int(N),
-                                          c_int(K), c_int(1 if up else 0), c_float(limit), c_float(alpha), _stream())
+                                          c_int(K), c_int(1 if up else 0), c_int(act), c_float(limit), c_float(alpha),
+                                          _stream())
             if st != -2:
                 _check(st, "moe_gemm_mma")
                 return
         _check(self._tl_moe_gemm(_ptr(a), c_int(a.stride(0)), _ptr(row_token), _ptr(w), _ptr(c), c_int(c.stride(0)),
-                                 _ptr(offsets), c_int(E), c_int(c.shape[0]), c_int(N), c_int(K), c_int(1 if up else 0),
+                                 _ptr(offsets), c_int(E), c_int(c.shape[0]), c_int(N), c_int(K), c_int(1 if up else 0), c_int(act),
                                  c_float(limit), c_float(alpha), _stream()), "moe_gemm")
 
     def moe_combine(self, yk: torch.Tensor, row_of: torch.Tensor, wt: torch.Tensor, h: torch.Tensor,
@@ -975,6 +1005,155 @@ class CoreOps:
         _check(self._tl_moe_combine(_ptr(yk), _ptr(row_of), _ptr(wt), _ptr(h), _ptr(out), c_int(out.stride(0)),
                                     c_int(T), c_int(H), c_int(top), c_int(1 if accumulate else 0), _stream()),
                "moe_combine")
+
+
+    # ---- a block whose sublayers run side by side ------------------------------------------------------
+    def close_block(self, x: torch.Tensor, experts=None, shared=None, add_rows: Optional[torch.Tensor] = None,
+                    add_vec: Optional[torch.Tensor] = None, w_next: Optional[torch.Tensor] = None,
+                    eps_next: float = 0.0, xn: Optional[torch.Tensor] = None) -> None:
+        """x[t] += sum_k wt[t, k] yk[row_of[t, k]] + sigmoid(sg[t]) ys[t] + add_rows[t] + add_vec, in place
+        (32-bit); with `w_next` (32-bit) also xn = x / rms(x) * w_next in the activation type.  `experts` =
+        (yk [pairs, H], row_of [T, top], wt [T, top]) or None; `shared` = (ys [T, H], sg [T] with any stride, or
+        None for a weight of one) or None."""
+        _need(x, torch.float32, "stream")
+        T, H = x.shape
+        yk = row_of = wt = ys = sg = None
+        top = 0
+        if experts is not None:
+            yk, row_of, wt = experts
+            _need(yk, torch.float32, "expert outputs")
+            _need(row_of, torch.int32, "rows")
+            _need(wt, torch.float32, "expert weights")
+            top = row_of.shape[1]
+            if yk.shape[1] != H or row_of.shape != (T, top) or wt.shape != (T, top):
+                raise KernelError("close_block: the experts' sizes do not match")
+        if shared is not None:
+            ys, sg = shared
+            _need(ys, torch.float32, "shared expert's output")
+            if sg is not None:
+                _need(sg, torch.float32, "shared expert's gate", contiguous=False)
+            if ys.shape != (T, H) or (sg is not None and sg.shape != (T,)):
+                raise KernelError("close_block: the shared expert's sizes do not match")
+        for t, what, n in ((add_rows, "rows to add", T * H), (add_vec, "vector to add", H), (w_next, "next norm's weight", H)):
+            if t is not None:
+                _need(t, torch.float32, what)
+                if t.numel() != n:
+                    raise KernelError(f"close_block: {what} have the wrong size")
+        if w_next is not None:
+            if xn is None or xn.shape != (T, H):
+                raise KernelError("close_block: the next norm needs a place for its result")
+            _need(xn, self.act_dtype, "normed stream")
+        _check(self._tl_close_block(_ptr(x), _ptr(yk), _ptr(row_of), _ptr(wt), c_int(top), _ptr(ys), _ptr(sg),
+                                    c_int(sg.stride(0) if sg is not None else 0), _ptr(add_rows), _ptr(add_vec),
+                                    _ptr(w_next), c_float(eps_next), _ptr(xn if w_next is not None else None), c_int(T),
+                                    c_int(H), _stream()), "close_block")
+
+    def qk_whole_norm_cache_write(self, z: torch.Tensor, bias: Optional[torch.Tensor], qw: torch.Tensor,
+                                  kw: torch.Tensor, eps: float, q_out: torch.Tensor, k_pages: torch.Tensor,
+                                  v_pages: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
+                                  seq_slot: torch.Tensor, page_table: torch.Tensor, nh: int, nkv: int, dim: int,
+                                  vdim: int) -> None:
+        """As `qk_norm_cache_write`, with one RMS norm over all query heads together and one over all key heads;
+        `qw` [nh * dim] and `kw` [nkv * dim] are their weights."""
+        _need(z, torch.float32, "projections", contiguous=False)
+        _need(q_out, self.act_dtype, "q out")
+        _need(k_pages, self.act_dtype, "k pages")
+        _need(v_pages, self.act_dtype, "v pages")
+        _need(page_table, torch.int32, "page table")
+        T = z.shape[0]
+        cols = (nh + nkv) * dim + nkv * vdim
+        if z.shape[1] < cols or z.stride(1) != 1 or q_out.shape != (T, nh * dim) or \
+                k_pages.shape[1:] != (nkv, PAGE, dim) or v_pages.shape[1:] != (nkv, vdim, PAGE):
+            raise KernelError("qk_whole_norm_cache_write: sizes do not match")
+        for t, n, what in ((bias, cols, "bias"), (qw, nh * dim, "q norm weight"), (kw, nkv * dim, "k norm weight")):
+            if t is not None:
+                _need(t, torch.float32, what)
+                if t.numel() != n:
+                    raise KernelError(f"qk_whole_norm_cache_write: {what} must have {n} entries")
+        _check(self._tl_qk_whole_norm_cache_write(
+            _ptr(z), c_int(z.stride(0)), _ptr(bias), _ptr(qw), _ptr(kw), c_float(eps), _ptr(q_out), _ptr(k_pages),
+            _ptr(v_pages), _ptr(token_pos), _ptr(token_seq), _ptr(seq_slot), _ptr(page_table),
+            c_int(page_table.stride(0)), c_int(T), c_int(nh), c_int(nkv), c_int(dim), c_int(vdim), _stream()),
+            "qk_whole_norm_cache_write")
+
+    # ---- state-space recurrence with one decay per head and token -----------------------------------------
+    def ssd_prep(self, z: torch.Tensor, col_x: int, col_dt: int, taps_w: torch.Tensor, bias: torch.Tensor,
+                 kept: torch.Tensor, xbc: torch.Tensor, dtla: torch.Tensor, neg_a: torch.Tensor,
+                 dt_bias: torch.Tensor, seq_start: torch.Tensor, seq_slot: torch.Tensor) -> None:
+        """From the 32-bit projections `z`: xbc [T, channels] = silu(conv(z[:, col_x:]) + bias) over `taps_w`
+        [channels, taps] (last column the current token's; inputs before the step come from `kept` [slots,
+        taps - 1, channels], oldest first, which then receives the step's last ones); dtla [T, H, 2] = (dt,
+        neg_a dt) with dt = softplus(z[:, col_dt:] + dt_bias)."""
+        _need(z, torch.float32, "projections", contiguous=False)
+        _need(xbc, self.act_dtype, "convolved channels")
+        for t, n in ((taps_w, "convolution taps"), (bias, "convolution bias"), (kept, "kept convolution inputs"),
+                     (dtla, "step sizes"), (neg_a, "decay rate"), (dt_bias, "step size bias")):
+            _need(t, torch.float32, n)
+        T, channels = xbc.shape
+        H, taps = neg_a.numel(), taps_w.shape[1]
+        if z.stride(1) != 1 or z.shape[0] != T or z.shape[1] < max(col_x + channels, col_dt + H) or \
+                taps_w.shape != (channels, taps) or bias.numel() != channels or kept.shape[1] < taps - 1 or \
+                kept.shape[2] != channels or (taps > 1 and kept.shape[1] != taps - 1) or dtla.shape != (T, H, 2) or \
+                dt_bias.numel() != H:
+            raise KernelError("ssd_prep: sizes do not match")
+        _check(self._tl_ssd_prep(_ptr(z), c_int(z.stride(0)), c_int(col_x), c_int(col_dt), _ptr(taps_w), _ptr(bias),
+                                 c_int(taps), _ptr(kept), _ptr(xbc), _ptr(dtla), _ptr(neg_a), _ptr(dt_bias),
+                                 _ptr(seq_start), _ptr(seq_slot), c_int(T), c_int(seq_slot.numel()), c_int(channels),
+                                 c_int(H), _stream()), "ssd_prep")
+
+    SSD_CHUNKED_FROM = 64     # tokens per sequence from which a step runs in chunks
+
+    def ssd_scan(self, xbc: torch.Tensor, dtla: torch.Tensor, D: torch.Tensor, state: torch.Tensor, y: torch.Tensor,
+                 seq_start: torch.Tensor, seq_slot: torch.Tensor, heads: int, groups: int, workspace=None,
+                 chunked: Optional[bool] = None) -> None:
+        """S <- exp(la) S + dt B x^T, y = S^T C + D x over each sequence's tokens of the step, from and into
+        `state` [slots, heads, N, P]; `xbc` = [x (heads P) | B (groups N) | C (groups N)] and `dtla` as
+        `ssd_prep` leaves them.  Long steps in bfloat16 run in chunks on the tensor cores (`chunked`: None
+        decides by the length; the same sums in another order)."""
+        _need(xbc, self.act_dtype, "convolved channels")
+        for t, n in ((dtla, "step sizes"), (D, "skip weights"), (state, "recurrent state"), (y, "recurrence out")):
+            _need(t, torch.float32, n)
+        T, channels = xbc.shape
+        B = seq_slot.numel()
+        N, P = int(state.shape[2]), int(state.shape[3])
+        if channels != heads * P + 2 * groups * N or dtla.shape != (T, heads, 2) or D.numel() != heads or \
+                state.shape[1] != heads or y.shape != (T, heads * P) or heads % groups:
+            raise KernelError("ssd_scan: sizes do not match")
+        if self.act_dtype == torch.bfloat16 and (chunked or (chunked is None and T >= self.SSD_CHUNKED_FROM * B)):
+            self.lib.tl_ssd_chunk_scratch.restype = c_longlong
+            n = int(self.lib.tl_ssd_chunk_scratch(c_int(T), c_int(B), c_int(heads), c_int(N), c_int(P)))
+            if n:
+                scratch = (workspace.get("ssd_chunks", (n,), torch.float32) if workspace is not None
+                           else torch.empty(n, dtype=torch.float32, device=xbc.device))
+                self.lib.tl_ssd_chunked.restype = c_int
+                st = self.lib.tl_ssd_chunked(_ptr(xbc), _ptr(dtla), _ptr(D), _ptr(state), _ptr(y), _ptr(seq_start),
+                                             _ptr(seq_slot), c_int(T), c_int(B), c_int(heads), c_int(groups), c_int(N),
+                                             c_int(P), c_int(channels), _ptr(scratch), c_int(_sm_count(xbc.device)),
+                                             _stream())
+                if st != -2:
+                    _check(st, "ssd_chunk_state")
+                    _check(0, "ssd_chunk_carry")
+                    _check(0, "ssd_chunk_out")
+                    return
+            if chunked:
+                raise KernelError("ssd_scan: the chunked form does not take these sizes")
+        _check(self._tl_ssd_walk(_ptr(xbc), _ptr(dtla), _ptr(D), _ptr(state), _ptr(y), _ptr(seq_start), _ptr(seq_slot),
+                                 c_int(B), c_int(heads), c_int(groups), c_int(N), c_int(P), c_int(channels), _stream()),
+               "ssd_walk")
+
+    def ssd_gate_norm(self, y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor,
+                      parts: int) -> None:
+        """out = g / rms(g) * w with g = y silu(z), the root mean square over each of `parts` equal parts of a
+        row; z 32-bit, rows may be strided."""
+        _need(y, torch.float32, "recurrence out")
+        _need(z, torch.float32, "gate", contiguous=False)
+        _need(w, torch.float32, "norm weight")
+        _need(out, self.act_dtype, "gated output")
+        T, inner = y.shape
+        if z.shape != (T, inner) or z.stride(1) != 1 or w.numel() != inner or out.shape != (T, inner) or inner % parts:
+            raise KernelError("ssd_gate_norm: sizes do not match")
+        _check(self._tl_ssd_gate_norm(_ptr(y), _ptr(z), c_int(z.stride(0)), _ptr(w), c_float(eps), _ptr(out), c_int(T),
+                                      c_int(inner), c_int(parts), _stream()), "ssd_gate_norm")
 
 
 class SamplingOps:

@@ -50,6 +50,8 @@ def expected_tensors(spec: ModelSpec) -> Dict[str, TensorSpec]:
             out.setdefault(f"{layer.prefix}.{name}", TensorSpec(tuple(shape), optional=True))
     out.update(lookup("norm", spec.final_norm.kind).expected_tensors(spec.final_norm,
                                                                      spec.final_norm_prefix))
+    if spec.pass_table_name is not None:
+        out[spec.pass_table_name] = TensorSpec((spec.pass_rows, spec.hidden_size))
     if not spec.tie_head_to_embedding:
         out[spec.head_name] = TensorSpec((spec.vocab_size, spec.hidden_size))
     return out
@@ -88,6 +90,7 @@ class DecoderModel:
                                  if spec.embedding_addend is not None else None)
         self.embedding: Optional[torch.Tensor] = None
         self.position_table: Optional[torch.Tensor] = None
+        self.pass_table: Optional[torch.Tensor] = None      # 32-bit: its rows join the stream
         self.head: Optional[torch.Tensor] = None
         # a part whose forward reads host-side values of the batch cannot be replayed from a
         # recorded graph; it says so by not setting `graph_safe`
@@ -111,6 +114,8 @@ class DecoderModel:
         self.embedding = self.rt.matrix(weights[self.spec.embedding_name])
         if self.spec.position_table_name is not None:
             self.position_table = self.rt.matrix(weights[self.spec.position_table_name])
+        if self.spec.pass_table_name is not None:
+            self.pass_table = weights[self.spec.pass_table_name].to(device=self.rt.device, dtype=torch.float32).contiguous()
         if self.embedding_addend is not None:
             self.embedding_addend.load(weights)
         for b in self.blocks:
@@ -129,7 +134,7 @@ class DecoderModel:
             if t is not None and t.data_ptr() not in seen:
                 seen.add(t.data_ptr())
                 total += t.numel() * t.element_size()
-        add(self.embedding); add(self.head); add(self.position_table)
+        add(self.embedding); add(self.head); add(self.position_table); add(self.pass_table)
         parts = [part for b in self.blocks for part in self._parts_of(b)]
         if self.embedding_addend is not None:
             parts.append(self.embedding_addend)
@@ -168,11 +173,23 @@ class DecoderModel:
         rt, ws = self.rt, self.rt.workspace
         T, H = batch.n_tokens, self.spec.hidden_size
         x = ws.get("stream", (T, H), torch.float32)
+        starts = self.spec.pass_starts
+        embedded = (ws.get("embedded", (T, H), torch.float32) if any(s.add_embedded for s in starts.values())
+                    else None)
+        # the embedding kernel keeps the copy and takes the first entry's addend along, unless something else
+        # joins the embedded tokens first
+        plain = self.embedding_addend is None
+        first = self._addend(starts.get(0), embedded)
+        vec = first[1] if plain and first is not None and first[0] is None else None
         rt.ops.embed(batch.tokens, self.embedding, x, batch.token_from, batch.token_src,
                      scale=self.spec.embedding_scale, position_table=self.position_table,
-                     token_pos=batch.token_pos)
-        if self.embedding_addend is not None:
+                     token_pos=batch.token_pos, copy=embedded if plain else None, add_vec=vec)
+        if not plain:
             self.embedding_addend.forward(batch, x)
+            if embedded is not None:
+                embedded.copy_(x)
+        if first is not None and vec is None:
+            rt.ops.close_block(x, None, None, *first)
         order = self.spec.order
         S = self.spec.streams
         if S is not None:
@@ -181,6 +198,13 @@ class DecoderModel:
         for k, i in enumerate(order):
             self.mixers[i].bind_cache(self.views[k])
             block = self.blocks[i]
+            addend = self._addend(starts.get(k + 1), embedded)
+            if addend is not None and not getattr(block, "takes_addend", False):
+                # nothing may be prepared from the stream before the addend has joined it
+                block.forward(x, batch, carry, None) if getattr(block, "takes_carry", False) else block.forward(x, batch)
+                rt.ops.close_block(x, None, None, *addend)
+                carry = None
+                continue
             if not getattr(block, "takes_carry", False):
                 block.forward(x, batch)       # the plain interface of a block
                 carry = None
@@ -189,12 +213,23 @@ class DecoderModel:
             # before it, and prepare the next block's: `first_norm` names the norm in question.
             nxt = self.blocks[order[k + 1]] if k + 1 < len(order) else None
             next_norm = getattr(nxt, "first_norm", None) if getattr(nxt, "takes_carry", False) else None
-            carry = block.forward(x, batch, carry, next_norm)
+            if addend is not None:
+                carry = block.forward(x, batch, carry, next_norm, addend=addend)
+            else:
+                carry = block.forward(x, batch, carry, next_norm)
         if batch.n_want == 0:
             return None
         xn = ws.get("head_normed", (batch.n_want, H), rt.act_dtype)
         self.final_norm(x, xn, rows=batch.want_rows)
         return self._head(batch, xn)
+
+    def _addend(self, start, embedded: Optional[torch.Tensor]):
+        """(rows, vector) that join the stream before an entry of the order, or None."""
+        if start is None:
+            return None
+        rows = embedded if start.add_embedded else None
+        vec = self.pass_table[start.row] if start.row is not None else None
+        return None if rows is None and vec is None else (rows, vec)
 
     def _forward_streams(self, batch, x: torch.Tensor, S: int) -> Optional[torch.Tensor]:
         """The layers over `S` residual streams [tokens, S, hidden], each of which starts as the embedded

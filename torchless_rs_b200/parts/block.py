@@ -247,3 +247,59 @@ class SandwichBlock:
 class SandwichMixerBlock(SandwichBlock):
     """The same block for a layer without a feed-forward: x <- x + N_1b(mixer(N_1(x)))."""
     norm_roles = ("mixer_norm", "mixer_out_norm")
+
+
+@register_block("parallel_sublayers")
+class ParallelSublayersBlock:
+    """x <- x + (mixer(h) + feed_forward(h)), h = N(x): one norm, both sublayers read its output.  Takes layers
+    with and without a feed-forward (part "none").
+
+    The mixer's output projection adds into the stream.  A feed-forward that offers `terms` leaves its last sum
+    to the block's closing kernel, which also takes what comes between this layer and the next (`addend`) and
+    the next norm, so the stream crosses memory once for all of them; any other feed-forward adds into the
+    stream itself.  Where the mixer can hold rows for the feed-forward in its input product (`take_rows`) and
+    the feed-forward names some (`input_rows`), both share that product.  The closing kernel takes next norms
+    with a 32-bit weight per coordinate (`weight`, `eps`)."""
+    norm_roles = ("norm",)
+    takes_carry = True
+    takes_addend = True
+
+    def __init__(self, spec, rt: Runtime, mixer, feed_forward, norms):
+        self.rt = rt
+        self.mixer = mixer
+        self.feed_forward = feed_forward
+        self.norms = dict(norms)
+        self.shares_input = hasattr(mixer, "take_rows") and hasattr(feed_forward, "input_rows")
+        if self.shares_input:
+            mixer.take_rows(feed_forward.input_rows())
+            feed_forward.own_input = False
+
+    @property
+    def first_norm(self):
+        return self.norms["norm"]
+
+    def forward(self, x: torch.Tensor, batch, carry=None, next_norm=None, addend=None):
+        """`addend` = (rows [tokens, hidden] or None, vector [hidden] or None): added to the stream after the
+        layer, before `next_norm`."""
+        rt, norm = self.rt, self.norms["norm"]
+        if isinstance(carry, NormedInput) and carry.norm is norm and carry.xn.shape == x.shape:
+            xn = carry.xn
+        else:
+            xn = norm(x, rt.workspace.get("block_normed", x.shape, rt.act_dtype))
+        self.mixer.forward(xn, x, batch)
+        experts = shared = None
+        if hasattr(self.feed_forward, "terms"):
+            experts, shared = self.feed_forward.terms(xn, batch, self.mixer.row_products if self.shares_input else None)
+        else:
+            self.feed_forward.forward(xn, x, batch)
+        w = getattr(next_norm, "weight", None)
+        fuse = w is not None and w.dtype == torch.float32 and w.numel() == x.shape[1]
+        if not fuse and experts is None and shared is None and addend is None:
+            return None
+        rows, vec = addend if addend is not None else (None, None)
+        if not fuse:
+            rt.ops.close_block(x, experts, shared, rows, vec)
+            return None
+        out = rt.workspace.get("block_normed", x.shape, rt.act_dtype)
+        rt.ops.close_block(x, experts, shared, rows, vec, w, next_norm.eps, out)
+        return NormedInput(out, next_norm)

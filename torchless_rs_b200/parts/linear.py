@@ -62,3 +62,33 @@ class Matmul:
         `GemmBf16.run` takes it): True if the tensor-core kernel took it, False if the caller has to
         run the product into 32-bit and the activation as a kernel of its own."""
         return self.fast is not None and self.fast.run(a, w, out, mode, act=act)
+
+
+class InputRows:
+    """For a mixer whose input goes through one stacked product into 32-bit: lets the feed-forward beside it,
+    which reads the same input, have rows of its own in that product (a router's, a gate's).
+
+    `take_rows(names)` (before `load`) names matrices to be stacked below the mixer's own;
+    `stack_input` makes the stacked matrix, `project_input` runs the product, and `row_products` is then the
+    [tokens, rows] view of what the taken rows gave, valid until the next product of this kind."""
+    row_names: tuple = ()
+    row_products = None
+
+    def take_rows(self, names) -> None:
+        self.row_names = tuple(names)
+
+    def stack_input(self, rt: Runtime, weights, own) -> torch.Tensor:
+        mats = list(own) + [weights[n] for n in self.row_names]
+        self.own_rows = sum(int(m.shape[0]) for m in own)
+        self.taken_rows = sum(int(weights[n].shape[0]) for n in self.row_names)
+        pad = -(self.own_rows + self.taken_rows) % 8       # rows of 32-bit results start on 16-byte boundaries
+        if pad:
+            mats.append(torch.zeros((pad, mats[0].shape[1]), dtype=mats[0].dtype, device=mats[0].device))
+        return rt.stack(mats)
+
+    def project_input(self, xn: torch.Tensor, name: str, T: int) -> torch.Tensor:
+        z = self.rt.workspace.get(name, (T, self.w_in.shape[0]), torch.float32)
+        self.matmul(xn, self.w_in, z, ops.MODE_STORE_F32)
+        if self.taken_rows:
+            self.row_products = z[:, self.own_rows:self.own_rows + self.taken_rows]
+        return z

@@ -10,7 +10,7 @@ The (token, expert) pairs are grouped by expert on the device; the experts' prod
 groups (no host value is read, so decode steps replay from CUDA graphs)."""
 from __future__ import annotations
 
-from typing import Dict
+from typing import Dict, Optional
 
 import torch
 
@@ -173,3 +173,97 @@ class GroupedSigmoidMoE:
                 self.matmul(xn, self.w_shared_up, zs, ops.MODE_STORE_F32)
                 rt.ops.clamped_glu(zs, self.shared_limit, self.gate_alpha, sact)
             self.matmul(sact, self.w_shared_down, residual, ops.MODE_ACCUM_F32)
+
+
+@register_feed_forward("moe_softmax_chosen")
+class SoftmaxChosenMoE:
+    """SwiGLU experts chosen by the router's logits and weighted by a softmax over the chosen alone, plus an
+    optional shared expert that every token uses, behind a sigmoid gate of its own.
+
+        z = W_router h + b (32-bit); the `top` largest z are chosen, with weights softmax over those z
+        expert(h) = W_down ( silu(W_gate h) * (W_up h) )
+        output = sum over the chosen of weight * expert(h)  +  sigmoid(W_sg h) * shared(h)
+
+    Parameters: `hidden_size`, `ff`, `experts`, `top`, `shared_ff` (None: no shared expert).  Tensors under the
+    prefix: e<i>.gate, e<i>.up, e<i>.down, router [experts, hidden], router.b, and with a shared expert
+    shared.gate, shared.up, shared.down, shared.sg [1, hidden].
+
+    `input_rows()` names the matrices whose 32-bit products with the input a mixer beside it may compute
+    (router, then the shared expert's gate); `terms(xn, batch, z)` then gives what a block's closing kernel adds
+    up: ((expert rows, rows of the choices, weights), (shared output, gate pre-activation) or None)."""
+    graph_safe = True
+    can_overwrite = True
+
+    def __init__(self, spec: PartSpec, prefix: str, rt: Runtime):
+        p = spec.params
+        self.hidden, self.ff = int(p["hidden_size"]), int(p["ff"])
+        self.experts, self.top = int(p["experts"]), int(p["top"])
+        self.shared_ff = int(p["shared_ff"]) if p.get("shared_ff") else None
+        if not 1 <= self.top <= self.experts:
+            raise ValueError("a token cannot choose more experts than there are")
+        self.prefix = prefix
+        self.rt = rt
+        self.matmul = Matmul(rt)
+        self.own_input = True         # False: a mixer computes the products of `input_rows`
+
+    @classmethod
+    def expected_tensors(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorSpec]:
+        p = spec.params
+        h, f, E = int(p["hidden_size"]), int(p["ff"]), int(p["experts"])
+        out = {f"{prefix}.router": TensorSpec((E, h), init=(h ** -0.5, 0.0)),
+               f"{prefix}.router.b": TensorSpec((E,), init=(0.1, 0.0))}
+        names = [(f"e{e}", f) for e in range(E)]
+        if p.get("shared_ff"):
+            names.append(("shared", int(p["shared_ff"])))
+            out[f"{prefix}.shared.sg"] = TensorSpec((1, h), init=(h ** -0.5, 0.0))
+        for n, width in names:
+            out[f"{prefix}.{n}.gate"] = TensorSpec((width, h), init=(h ** -0.5, 0.0))
+            out[f"{prefix}.{n}.up"] = TensorSpec((width, h), init=(h ** -0.5, 0.0))
+            out[f"{prefix}.{n}.down"] = TensorSpec((h, width), init=(width ** -0.5, 0.0))
+        return out
+
+    def input_rows(self):
+        return [f"{self.prefix}.router"] + ([f"{self.prefix}.shared.sg"] if self.shared_ff else [])
+
+    def load(self, weights: Dict[str, torch.Tensor]) -> None:
+        p, rt, E = self.prefix, self.rt, self.experts
+        self.w_up = rt.stack([weights[f"{p}.e{e}.{n}"] for e in range(E) for n in ("gate", "up")]) \
+            .view(E, 2 * self.ff, self.hidden)
+        self.w_down = rt.stack([weights[f"{p}.e{e}.down"] for e in range(E)]).view(E, self.hidden, self.ff)
+        self.router_b = weights[f"{p}.router.b"].to(device=rt.device, dtype=torch.float32).contiguous()
+        if self.own_input:
+            self.w_rows = rt.stack([weights[n] for n in self.input_rows()])
+        if self.shared_ff:
+            self.w_shared_up = rt.stack([weights[f"{p}.shared.gate"], weights[f"{p}.shared.up"]])
+            self.w_shared_down = rt.matrix(weights[f"{p}.shared.down"])
+
+    def terms(self, xn: torch.Tensor, batch, z: Optional[torch.Tensor] = None):
+        rt, ws = self.rt, self.rt.workspace
+        T, E, top = xn.shape[0], self.experts, self.top
+        if z is None:
+            z = ws.get("moe_logits", (T, self.w_rows.shape[0]), torch.float32)
+            self.matmul(xn, self.w_rows, z, ops.MODE_STORE_F32)
+        idx = ws.get("moe_idx", (T, top), torch.int32)
+        wt = ws.get("moe_wt", (T, top), torch.float32)
+        rt.ops.moe_route_chosen(z[:, :E], self.router_b, top, idx, wt)
+        offsets = ws.get("moe_offsets", (E + 1,), torch.int32)
+        row_token = ws.get("moe_row_token", (T * top,), torch.int32)
+        row_of = ws.get("moe_row_of", (T, top), torch.int32)
+        rt.ops.moe_plan(idx, E, offsets, row_token, row_of)
+        yk = ws.get("moe_expert_out", (T * top, self.hidden), torch.float32)
+        act = ws.get("moe_act", (T * top, self.ff), rt.act_dtype)
+        rt.ops.moe_gemm(xn, row_token, self.w_up, act, offsets, up=True, act=ops.ACT_PLAIN)
+        rt.ops.moe_gemm(act, None, self.w_down, yk, offsets, up=False)
+        if not self.shared_ff:
+            return (yk, row_of, wt), None
+        sact = ws.get("moe_shared_act", (T, self.shared_ff), rt.act_dtype)
+        self.matmul(xn, self.w_shared_up, sact, ops.MODE_SWIGLU)
+        ys = ws.get("moe_shared_out", (T, self.hidden), torch.float32)
+        self.matmul(sact, self.w_shared_down, ys, ops.MODE_STORE_F32)
+        return (yk, row_of, wt), (ys, z[:, E])
+
+    def forward(self, xn: torch.Tensor, residual: torch.Tensor, batch, emit=None, overwrite: bool = False) -> None:
+        experts, shared = self.terms(xn, batch)
+        if overwrite:
+            residual.zero_()
+        self.rt.ops.close_block(residual, experts, shared)

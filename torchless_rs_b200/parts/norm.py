@@ -75,14 +75,16 @@ class ScalarRMSNorm:
 @register_norm("rmsnorm_one_plus")
 class OnePlusRMSNorm:
     """y = x / sqrt(mean(x^2) + eps) * (1 + w): the stored weight lies around zero.  Parameters:
-    `size`, `eps`.  Its tensor is stored under the norm's own name (no `.weight`).  `weight` is
-    the 32-bit factor 1 + w, which is what the row kernel and the stream kernels multiply by."""
+    `size`, `eps`; optionally `output_scale`, a constant factor on y (for a final norm: a factor on the
+    logits, since the head is linear).  Its tensor is stored under the norm's own name (no `.weight`).
+    `weight` is the 32-bit factor 1 + w, which is what the row kernel and the stream kernels multiply by."""
 
     foldable = False
 
     def __init__(self, spec: PartSpec, prefix: str, rt: Runtime):
         self.size = int(spec.params["size"])
         self.eps = float(spec.params["eps"])
+        self.output_scale = float(spec.params.get("output_scale", 1.0))
         self.name = prefix
         self.rt = rt
         self.weight: Optional[torch.Tensor] = None
@@ -93,7 +95,7 @@ class OnePlusRMSNorm:
 
     def load(self, weights: Dict[str, torch.Tensor]) -> None:
         w = weights[self.name].to(device=self.rt.device, dtype=torch.float32)
-        self.weight = (w + 1.0).contiguous()
+        self.weight = ((w + 1.0) * self.output_scale).contiguous()
 
     def __call__(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         self.rt.ops.rmsnorm(x, self.weight, self.eps, out, rows)
