@@ -765,7 +765,7 @@ def test_tensor_memory_attention_takes_caps_and_windows(H, G, dim, rot, window, 
             step, view = _Step(pages, first, last), _View(pages)
             qs = q[first:last + 1].contiguous()
             if cap:
-                assert fast.run_capped(qs, view, out, step, H, G, window, scale, cap), "the kernel did not take the step"
+                assert fast.run_prompt(qs, view, out, step, H, G, window, scale, cap), "the kernel did not take the step"
             else:
                 fast.prefill(qs, view.k_pages, view.v_pages, out, step.seq_start, step.seq_len, step.seq_slot,
                              view.page_table, 1, step.max_new, H, G, window, scale, variant="tc")

@@ -135,8 +135,8 @@ class AttentionBf16:
                 self._prefill_tma.restype = c_int
                 self._prefill_tc = getattr(self.lib, f"tl_attn_prefill_tc_hd{head_dim}")
                 self._prefill_tc.restype = c_int
-                self._prefill_tc_cap = getattr(self.lib, f"tl_attn_prefill_tc_cap_hd{head_dim}")
-                self._prefill_tc_cap.restype = c_int
+                self._prefill_tc_any = getattr(self.lib, f"tl_attn_prefill_tc_any_hd{head_dim}")
+                self._prefill_tc_any.restype = c_int
                 self._tc_error = getattr(self.lib, f"tl_attn_tc_take_error_hd{head_dim}")
                 self._tc_error.restype = c_int
                 self._tma_error = getattr(self.lib, f"tl_attn_tma_take_error_hd{head_dim}")
@@ -225,24 +225,37 @@ class AttentionBf16:
                              c_int(nkv), c_int(window or 0), c_float(scale), _stream()),
                "attn_prefill")
 
-    def run_capped(self, q, cache_view, out, batch, nh, nkv, window, scale, cap) -> bool:
-        """A prompt step whose scores are capped, s <- cap tanh(s scale / cap), on the tensor-memory kernel.
-        False where that kernel does not take the step (decode steps, few new tokens, other head sizes):
-        the caller then uses a kernel that does."""
-        if getattr(self, "_prefill_tc_cap", None) is None or nh // nkv > MAX_GROUP or batch.is_decode or \
-                batch.max_new < 128:
+    # New tokens of a sequence from which a step's prompts run on the tensor-memory kernel.
+    TC_FROM = 128
+
+    @staticmethod
+    def takes_prompts(dim: int, vdim: int, group: int) -> bool:
+        """Whether the tensor-memory prompt kernel takes these sizes."""
+        return dim == vdim and dim in FAST_HEAD_DIMS and dim % 64 == 0 and group <= MAX_GROUP
+
+    def run_prompt(self, q, cache_view, out, batch, nh, nkv, window, scale, cap=None, sink=None) -> bool:
+        """A prompt step on the tensor-memory kernel, with capped scores (s <- cap tanh(s scale / cap)) and / or a
+        sink (32-bit, one logit per head, in the denominator only).  False where that kernel does not take
+        the step (decode steps, few new tokens, other head sizes): the caller then uses a kernel that does."""
+        if getattr(self, "_prefill_tc_any", None) is None or nh // nkv > MAX_GROUP or batch.is_decode or \
+                batch.max_new < self.TC_FROM or not scale > 0:
             return False
         c = cache_view
         for t, n in ((q, "q"), (c.k_pages, "k pages"), (c.v_pages, "v pages"), (out, "out")):
             _need(t, torch.bfloat16, f"attn prefill {n}")
-        st = self._prefill_tc_cap(_ptr(q), c_longlong(q.shape[0]), _ptr(c.k_pages), _ptr(c.v_pages),
+        if sink is not None:
+            _need(sink, torch.float32, "attn prefill sink")
+            if sink.numel() != nh:
+                raise KernelError("attn prefill: one sink per head is needed")
+        st = self._prefill_tc_any(_ptr(q), c_longlong(q.shape[0]), _ptr(c.k_pages), _ptr(c.v_pages),
                                   c_longlong(c.k_pages.shape[0]), _ptr(out), _ptr(batch.seq_start),
                                   _ptr(batch.seq_len), _ptr(batch.seq_slot), _ptr(c.page_table),
                                   c_int(c.page_table.stride(0)), c_int(batch.n_seqs), c_int(batch.max_new), c_int(nh),
-                                  c_int(nkv), c_int(window or 0), c_float(scale), c_float(cap), _stream())
+                                  c_int(nkv), c_int(window or 0), c_float(scale), c_float(cap or 0.0), _ptr(sink),
+                                  _stream())
         if st == -2:
             return False
-        _check(st, "attn_prefill_tc_cap")
+        _check(st, "attn_prefill_tc_cap" if cap else "attn_prefill_tc_sink")
         return True
 
     def run(self, q, cache_view, out, batch, nh, nkv, window, scale, workspace) -> bool:

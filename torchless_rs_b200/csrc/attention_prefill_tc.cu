@@ -190,6 +190,8 @@ __device__ __forceinline__ uint32_t tc_idesc(int n) {   // bf16 x bf16 -> f32, M
 // CAP: the scaled scores are capped, s <- cap tanh(s scale / cap), before mask and softmax; `scale_log2` is
 // then log2(e) alone, `cap_c2` = 2 log2(e) scale / cap, and tanh(x) = 1 - 2 / (e^(2x) + 1) by one fast
 // exponential and a reciprocal by Newton steps (absolute error about 1e-7; exact at both ends).
+// `sink` (null: none): a logit per head that is in the softmax's denominator and has no value; it opens every
+// row's reference and sum.
 template <bool CAP>
 __global__ void __launch_bounds__(TC_THREADS)
 FN(attn_prefill_tc_kernel)(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
@@ -197,7 +199,7 @@ FN(attn_prefill_tc_kernel)(const __grid_constant__ CUtensorMap tm_q, const __gri
                            const int* __restrict__ seq_start, const int* __restrict__ seq_len,
                            const int* __restrict__ seq_slot, const int* __restrict__ page_table,
                            int table_stride, int nh, int nkv, int window, float scale_log2, float cap,
-                           float cap_c2) {
+                           float cap_c2, const float* __restrict__ sink) {
   // The tiles need 1024-byte alignment (128-byte swizzle) and two blocks per SM leave no room
   // for padding, so the dynamic shared memory itself must start on such a boundary (it does
   // when the kernel has no static shared memory; checked below).
@@ -350,7 +352,8 @@ FN(attn_prefill_tc_kernel)(const __grid_constant__ CUtensorMap tm_q, const __gri
     const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     const uint32_t t_s = tmem_base + ((uint32_t)(warp * 32) << 16);
     const uint32_t t_o = tmem_o + ((uint32_t)(warp * 32) << 16);
-    float m = -INFINITY, l = 0.0f;
+    float m = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
+    float l = sink != nullptr ? 1.0f : 0.0f;
     bool ok = true;
     for (int i = 0; i < n_pg; ++i) {
       ok = tc_mbar_wait(&s_full[i & 1], (uint32_t)(i >> 1) & 1u, abort_flag, 5);
@@ -540,12 +543,12 @@ static bool tc_make_map(CUtensorMap* map, const void* ptr, long long rows, long 
 
 // q, out [T, nh*HEAD_DIM]; max_new = the most new tokens any sequence of the step has.
 // Returns -2 for sizes this kernel does not take.
-// `cap` > 0: scores are capped, s <- cap tanh(s scale / cap).
-extern "C" int FN(tl_attn_prefill_tc_cap)(const void* q, long long T, const void* k_pages, const void* v_pages,
+// `cap` > 0: scores are capped, s <- cap tanh(s scale / cap).  `sink`: a logit per head, or null.
+extern "C" int FN(tl_attn_prefill_tc_any)(const void* q, long long T, const void* k_pages, const void* v_pages,
                                           long long n_pages, void* out, const int* seq_start,
                                           const int* seq_len, const int* seq_slot, const int* page_table,
                                           int table_stride, int B, int max_new, int nh, int nkv, int window,
-                                          float scale, float cap, cudaStream_t stream) {
+                                          float scale, float cap, const float* sink, cudaStream_t stream) {
 #if HEAD_DIM % 64 != 0
   return -2;
 #else
@@ -574,10 +577,10 @@ extern "C" int FN(tl_attn_prefill_tc_cap)(const void* q, long long T, const void
   if (cap > 0.0f)
     return tl_launch(FN(attn_prefill_tc_kernel)<true>, grid, dim3(TC_THREADS), smem, stream, tq, tk, tv,
                      (__nv_bfloat16*)out, seq_start, seq_len, seq_slot, page_table, table_stride, nh, nkv,
-                     window, log2e, cap, 2.0f * log2e * scale / cap);
+                     window, log2e, cap, 2.0f * log2e * scale / cap, sink);
   return tl_launch(FN(attn_prefill_tc_kernel)<false>, grid, dim3(TC_THREADS), smem, stream, tq, tk, tv,
                    (__nv_bfloat16*)out, seq_start, seq_len, seq_slot, page_table, table_stride, nh, nkv,
-                   window, scale * log2e, 0.0f, 0.0f);
+                   window, scale * log2e, 0.0f, 0.0f, sink);
 #endif
 }
 
@@ -586,8 +589,8 @@ extern "C" int FN(tl_attn_prefill_tc)(const void* q, long long T, const void* k_
                                       const int* seq_len, const int* seq_slot, const int* page_table,
                                       int table_stride, int B, int max_new, int nh, int nkv, int window,
                                       float scale, cudaStream_t stream) {
-  return FN(tl_attn_prefill_tc_cap)(q, T, k_pages, v_pages, n_pages, out, seq_start, seq_len, seq_slot, page_table,
-                                    table_stride, B, max_new, nh, nkv, window, scale, 0.0f, stream);
+  return FN(tl_attn_prefill_tc_any)(q, T, k_pages, v_pages, n_pages, out, seq_start, seq_len, seq_slot, page_table,
+                                    table_stride, B, max_new, nh, nkv, window, scale, 0.0f, nullptr, stream);
 }
 
 extern "C" int FN(tl_attn_tc_take_error)() {

@@ -597,7 +597,7 @@ def rupasun_kernels(size: str, T: int, B: int, ctx: int, iters: int, file=None) 
             fast = AttentionBf16.get(width) if width == vdim and width in (32, 64, 128) else None
             if fast is not None and cap is None and fast.run(qq, view, oo, _B, heads, G, window, scale, ws):
                 return
-            if fast is not None and cap is not None and fast.run_capped(qq, view, oo, _B, heads, G, window, scale, cap):
+            if fast is not None and cap is not None and fast.run_prompt(qq, view, oo, _B, heads, G, window, scale, cap):
                 return
             run_attention(o, qq, kk, vv, None, None, oo, pos, seq, slot, table, heads, G, width, vdim, window, 0, scale,
                           cap, _B, ws)
@@ -916,6 +916,214 @@ def fezolorn_kernels(size: str, T: int, B: int, ctx: int, iters: int, file=None)
     return rows
 
 
+# Layer sizes at which the Dunesun kernels are measured: the width, heads and feed-forward of a 1B- and a
+# 7B-class decoder; attention with a quarter as many key/value heads and a window of 4096, and a state-space
+# layer of twice the width (heads of 64, a state of 128 entries per head, four taps) in turn; sixteen experts
+# of which four are chosen, and a shared one, in every layer.
+DUNESUN_SIZES = {
+    "1b": dict(width=2048, heads=16, kv_heads=4, dim=128, window=4096, m_heads=64, m_vdim=64, m_state=128, m_groups=1,
+               conv=4, norm_groups=1, experts=16, top=4, e_ff=1408, vocab=32000),
+    "7b": dict(width=4096, heads=32, kv_heads=8, dim=128, window=4096, m_heads=128, m_vdim=64, m_state=128, m_groups=8,
+               conv=4, norm_groups=8, experts=16, top=4, e_ff=3584, vocab=32000),
+}
+
+
+def dunesun_config(size: str, layers: int) -> dict:
+    """config.json of a Dunesun model of `layers` layers at these sizes: the two mixers in turn."""
+    z = DUNESUN_SIZES[size]
+    mlp = {"kind": "moe", "expert": {"ff": z["e_ff"]}, "router": {"experts": z["experts"], "top": z["top"]},
+           "shared": {"ff": z["e_ff"]}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"],
+        "scale": 1.0 / math.sqrt(z["dim"]), "mask": {"size": z["window"]}}}
+    ssm = {"type": "mamba2", "mlp": mlp, "mixer": {
+        "heads": z["m_heads"], "vdim": z["m_vdim"], "state": z["m_state"], "groups": z["m_groups"], "conv": z["conv"],
+        "norm_groups": z["norm_groups"]}}
+    return {"architecture": "Dunesun", "width": z["width"], "vocab": z["vocab"], "norm": {"eps": 1e-5},
+            "logit_scale": 0.5, "max_positions": 8192, "layers": [(ssm, att)[i % 2] for i in range(layers)]}
+
+
+def dunesun_like(size: str, layers: int) -> dict:
+    """The closest existing model at equal size: the fourth design with its windowed attention and its experts
+    (as many, as wide, as many chosen, one shared) in every layer."""
+    z = DUNESUN_SIZES[size]
+    win = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": 1.0,
+           "softcap": 50.0, "mask": {"size": z["window"]}, "rot": {"dims": z["dim"] // 2, "base": 10000.0}}
+    moe = {"kind": "moe", "expert": {"ff": z["e_ff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": 4, "keep": 2}},
+           "shared": {"ff": z["e_ff"], "limit": 7.0}}
+    return {"architecture": "Rupasun", "width": z["width"], "vocab": z["vocab"], "norm": {"eps": 1e-5},
+            "max_position_embeddings": 32768,
+            "layers": [{"type": "attention_2", "mixer": win, "mlp": moe} for _ in range(layers)]}
+
+
+def dunesun_kernels(size: str, T: int, B: int, ctx: int, iters: int, file=None) -> list:
+    """Every kernel that the Dunesun design added or changed, alone at the sizes `size`, for a prompt of T tokens
+    and for a decode step of B sequences at a context of `ctx`, beside the like kernel of an existing model at
+    equal sizes.  Rows and roofline as `kikopel_kernels` defines them."""
+    import json
+    import os
+    from .csrc import ops
+    from .csrc.attention_bf16 import AttentionBf16
+    from .parts.runtime import Workspace
+    from .parts.sink_attention import run_attention
+    z = DUNESUN_SIZES[size]
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    pk = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
+    if os.path.isfile(pk):
+        peaks.update(json.load(open(pk)))
+    o = ops.core_ops(torch.bfloat16)
+    dev, bf = "cuda", torch.bfloat16
+    H, G, dim, W = z["heads"], z["kv_heads"], z["dim"], z["width"]
+    rows = []
+
+    def report(name, case, us, byts, flops):
+        t_mem, t_fl = byts / (peaks["hbm_gbs"] * 1e3), flops / (peaks["bf16_tflops"] * 1e6)     # microseconds
+        frac = max(t_mem, t_fl) / us
+        rows.append({"kernel": name, "case": case, "us": round(us, 2), "roofline_frac": round(frac, 4),
+                     "bound": "memory" if t_mem >= t_fl else "tensor"})
+        print(f"{name:38s} {case:22s} {us:10.2f} us   {frac:7.4f} of the roofline ({rows[-1]['bound']})", file=file)
+
+    ws = Workspace(torch.device("cuda"))
+    for case, n_tok, seqs, past in ((f"prompt {T}", T, 1, 0), (f"decode {B} x {ctx}", B, B, ctx - 1)):
+        per = n_tok // seqs
+        few = max(2, iters // 8) if n_tok > 64 else iters
+        pos = torch.cat([torch.arange(past, past + per, dtype=torch.int32) for _ in range(seqs)]).to(dev)
+        seq = torch.arange(seqs, dtype=torch.int32).repeat_interleave(per).to(dev)
+        start = (torch.arange(seqs + 1, dtype=torch.int32) * per).to(dev)
+        seen = sum(min(p + 1, z["window"]) for p in range(past, past + per)) * seqs
+        kp, vp, table, slot = _paged(seqs, past + per, G, dim)
+        lens = torch.full((seqs,), past + per, dtype=torch.int32, device=dev)
+        # --- attention with a sink, beside the closest model's capped window attention
+        q = torch.randn((n_tok, H * dim), device=dev, dtype=bf)
+        out = torch.empty((n_tok, H * dim), device=dev, dtype=bf)
+        sink = torch.zeros(H, device=dev)
+        fast = AttentionBf16.get(dim)
+
+        class _B:      # what the kernel choice reads of a step
+            n_tokens, n_seqs, is_decode, max_len, seq_start, seq_len, seq_slot, max_new = \
+                n_tok, seqs, per == 1, past + per, start, lens, slot, per
+
+        class _C:      # the cache view of the attention kernels
+            k_pages, v_pages, page_table = kp, vp, table
+
+        def attend(sk, cap):
+            if not fast.run_prompt(q, _C, out, _B, H, G, z["window"], 0.088, cap=cap, sink=sk):
+                run_attention(o, q, kp, vp, None, sk, out, pos, seq, slot, table, H, G, dim, dim, z["window"], 0, 0.088,
+                              cap, _B, ws)
+        cache_b = 2.0 * seqs * min(past + per, z["window"]) * G * 2 * dim
+        us = _time(lambda: attend(sink, None), few)
+        report("attention (window, sink)", case, us, cache_b + n_tok * H * dim * 4.0, 4.0 * H * dim * seen)
+        us = _time(lambda: attend(None, 50.0), few)
+        report("  like: attention (window, cap)", case, us, cache_b + n_tok * H * dim * 4.0, 4.0 * H * dim * seen)
+        # --- norm over the whole projection and cache write, beside the norm per head
+        cols = (H + 2 * G) * dim
+        zq = torch.randn((n_tok, cols), device=dev)
+        qw, kw = torch.ones(H * dim, device=dev), torch.ones(G * dim, device=dev)
+        us = _time(lambda: o.qk_whole_norm_cache_write(zq, None, qw, kw, 1e-5, q, kp, vp, pos, seq, slot, table, H, G,
+                                                       dim, dim), iters)
+        report("qk_whole_norm_cache_write", case, us, n_tok * cols * 6.0, 0.0)
+        hw = torch.ones(dim, device=dev)
+        us = _time(lambda: o.qk_norm_cache_write(zq, None, hw, hw, 1e-5, q, kp, vp, pos, seq, slot, table, H, G, dim,
+                                                 dim), iters)
+        report("  like: qk_norm_cache_write", case, us, n_tok * cols * 6.0, 0.0)
+        # --- the state-space layer: preparation, recurrence, gate and norm
+        mh, mg, N, P, taps = z["m_heads"], z["m_groups"], z["m_state"], z["m_vdim"], z["conv"]
+        inner = mh * P
+        ch = inner + 2 * mg * N
+        zz = torch.randn((n_tok, inner + ch + mh), device=dev)
+        xbc = torch.empty((n_tok, ch), device=dev, dtype=bf)
+        dtla = torch.empty((n_tok, mh, 2), device=dev)
+        kept = torch.zeros((seqs, taps - 1, ch), device=dev)
+        tw, cb = torch.randn((ch, taps), device=dev), torch.zeros(ch, device=dev)
+        na, dtb, D = -torch.ones(mh, device=dev), torch.zeros(mh, device=dev), torch.ones(mh, device=dev)
+        state = torch.zeros((seqs, mh, N, P), device=dev)
+        so = torch.empty((n_tok, inner), device=dev)
+        us = _time(lambda: o.ssd_prep(zz, inner, inner + ch, tw, cb, kept, xbc, dtla, na, dtb, start, slot), iters)
+        report("ssd_prep", case, us, n_tok * (ch * 6.0 + mh * 12.0) + seqs * (taps - 1) * ch * 8.0, 0.0)
+        us = _time(lambda: o.ssd_scan(xbc, dtla, D, state, so, start, slot, mh, mg, workspace=ws), few)
+        report("ssd_scan", case, us, n_tok * (ch * 2.0 + mh * 8.0 + inner * 4.0) + seqs * mh * N * P * 8.0,
+               4.0 * n_tok * mh * N * P)
+        gated = torch.empty((n_tok, inner), device=dev, dtype=bf)
+        nw = torch.ones(inner, device=dev)
+        us = _time(lambda: o.ssd_gate_norm(so, zz[:, :inner], nw, 1e-5, gated, z["norm_groups"]), iters)
+        report("ssd_gate_norm", case, us, n_tok * inner * 10.0, 0.0)
+        # the like kernels: the delta rule's preparation at as many channels, gated linear attention at the same
+        # state in heads of 64 x 128, the norm over the concatenated heads with its gate
+        rd, rv = 64, 128
+        rh = mh * N * P // (rd * rv)
+        rg = max(1, rh // 2)
+        C = 2 * rg * rd + rh * rv
+        y = torch.empty((n_tok, C), device=dev)
+        gates = torch.empty((n_tok, 2 * rh + rg), device=dev)
+        kept2 = torch.zeros((seqs, taps - 1, C), device=dev)
+        tw2, na2, dtb2 = torch.randn((C, taps), device=dev), -torch.ones(rh, device=dev), torch.zeros(rh, device=dev)
+        z2 = torch.randn((n_tok, C + 2 * rh), device=dev)
+
+        def prep():
+            o.delta_prep(z2, tw2, kept2, y, gates, na2, dtb2, C, C + rh, seq, start, slot, rg, rh, rd, rv, 1e-6, 0.125)
+            o.conv_state_update(z2, kept2, start, slot, C)
+        us = _time(prep, iters)
+        report("  like: delta_prep + state update", case, us, n_tok * (C * 8.0 + (4 * rh + rg) * 4.0) + seqs * (taps - 1) * C * 8.0, 0.0)
+        hd, hv = rh * rd, rh * rv
+        z3 = torch.randn((n_tok, 2 * hd + 2 * hv), device=dev)
+        za = torch.randn((n_tok, hd), device=dev) + 3.0
+        ab = torch.zeros(hd, device=dev)
+        state3 = torch.zeros((seqs, rh, rd, rv), device=dev)
+        so3 = torch.empty((n_tok, hv), device=dev)
+        us = _time(lambda: o.gla_scan(z3[:, :hd], z3[:, hd:2 * hd], z3[:, 2 * hd:2 * hd + hv], za, ab, 16.0, 0.125,
+                                      state3, so3, start, slot, rh, rd, rv, workspace=ws), few)
+        report("  like: gla_scan (equal state)", case, us, n_tok * (3 * hd + 2 * hv) * 4.0 + seqs * hd * rv * 8.0,
+               4.0 * n_tok * hd * rv)
+        gated3 = torch.empty((n_tok, inner), device=dev, dtype=bf)
+        us = _time(lambda: o.headnorm_silu_gate(so, nw, 1e-6, zz[:, :inner], gated3, 1, inner), iters)
+        report("  like: headnorm gate (one wide head)", case, us, n_tok * inner * 10.0, 0.0)
+        del z3, za, z2, y
+        # --- the experts: choice and grouping, the grouped products; the closing kernel
+        E, top, f = z["experts"], z["top"], z["e_ff"]
+        zr = torch.randn((n_tok, E + 1), device=dev)
+        idx = torch.empty((n_tok, top), dtype=torch.int32, device=dev)
+        wt = torch.empty((n_tok, top), device=dev)
+        rb = torch.zeros(E, device=dev)
+        off = torch.empty(E + 1, dtype=torch.int32, device=dev)
+        row_token = torch.empty(n_tok * top, dtype=torch.int32, device=dev)
+        row_of = torch.empty((n_tok, top), dtype=torch.int32, device=dev)
+        us = _time(lambda: o.moe_route_chosen(zr[:, :E], rb, top, idx, wt), iters)
+        report("moe_route_chosen", case, us, n_tok * (E * 4.0 + top * 8.0), 0.0)
+        us = _time(lambda: o.moe_route_grouped(zr[:, :E], 4, 2, top, 2.5, idx, wt), iters)
+        report("  like: moe_route_grouped", case, us, n_tok * (E * 4.0 + top * 8.0), 0.0)
+        o.moe_route_chosen(zr[:, :E], rb, top, idx, wt)
+        us = _time(lambda: o.moe_plan(idx, E, off, row_token, row_of), iters)
+        report("moe_plan (shared with the like model)", case, us, n_tok * top * 12.0, 0.0)
+        xn = torch.randn((n_tok, W), device=dev, dtype=bf)
+        w_up = torch.randn((E, 2 * f, W), device=dev, dtype=bf) * 0.02
+        w_dn = torch.randn((E, W, f), device=dev, dtype=bf) * 0.02
+        act = torch.empty((n_tok * top, f), device=dev, dtype=bf)
+        yk = torch.empty((n_tok * top, W), device=dev)
+        pairs = n_tok * top
+        used = int((off[1:] > off[:-1]).sum())         # experts whose matrices this step reads
+        up_b, up_f = used * 2 * f * W * 2.0 + pairs * (W + f) * 2.0, 4.0 * pairs * f * W
+        us = _time(lambda: o.moe_gemm(xn, row_token, w_up, act, off, up=True, act=ops.ACT_PLAIN), few)
+        report("moe_gemm (gate, up, silu)", case, us, up_b, up_f)
+        us = _time(lambda: o.moe_gemm(xn, row_token, w_up, act, off, up=True, limit=7.0, alpha=1.702), few)
+        report("  like: moe_gemm (clamped)", case, us, up_b, up_f)
+        us = _time(lambda: o.moe_gemm(act, None, w_dn, yk, off, up=False), few)
+        report("moe_gemm (down, as the like model's)", case, us, used * f * W * 2.0 + pairs * (f * 2.0 + W * 4.0), 2.0 * pairs * f * W)
+        x, ys, rows_ = (torch.randn((n_tok, W), device=dev) for _ in range(3))
+        vec, w32 = torch.ones(W, device=dev), torch.ones(W, device=dev)
+        us = _time(lambda: o.close_block(x, (yk, row_of, wt), (ys, zr[:, E]), None, None, w32, 1e-5, xn), iters)
+        report("close_block (experts, shared, norm)", case, us, n_tok * W * (4.0 * top + 14.0), 0.0)
+        us = _time(lambda: o.close_block(x, (yk, row_of, wt), (ys, zr[:, E]), rows_, vec, w32, 1e-5, xn), iters)
+        report("close_block (and a pass's start)", case, us, n_tok * W * (4.0 * top + 18.0), 0.0)
+
+        def like_close():
+            o.moe_combine(yk, row_of, wt, xn, x, accumulate=False)
+            o.norm_add_norm(ys, w32, 1e-5, x, w32, 1e-5, xn)
+        us = _time(like_close, iters)
+        report("  like: moe_combine + norm_add_norm", case, us, n_tok * W * (4.0 * top + 18.0), 0.0)
+    return rows
+
+
 def step(B: int, context: int, prefill: int, layers: int, iters: int) -> None:
     from . import from_random
     from .config import config_from_dict
@@ -1078,15 +1286,16 @@ def timeline(B: int, context: int, layers: int) -> None:
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("what", choices=["gemm", "attn-decode", "attn-prefill", "elementwise", "step", "timeline", "decode",
-                                     "kikopel-kernels", "tovapel-kernels", "rupasun-kernels", "fezolorn-kernels"])
+                                     "kikopel-kernels", "tovapel-kernels", "rupasun-kernels", "fezolorn-kernels",
+                                     "dunesun-kernels"])
     ap.add_argument("sizes", type=int, nargs="+")
     ap.add_argument("--iters", type=int, default=50)
     ap.add_argument("--layers", type=int, default=4, help="layers of the model that `step` builds")
     ap.add_argument("--model", default="mistral7b", choices=sorted(MODEL_SIZES),
                     help="step, timeline: whose layer sizes the model has")
     ap.add_argument("--kikopel-size", default="1b", choices=sorted(KIKOPEL_SIZES),
-                    help="kikopel-kernels / tovapel-kernels / rupasun-kernels / fezolorn-kernels TOKENS BATCH CONTEXT: whose layer sizes "
-                         "the kernels get")
+                    help="kikopel-kernels / tovapel-kernels / rupasun-kernels / fezolorn-kernels / dunesun-kernels "
+                         "TOKENS BATCH CONTEXT: whose layer sizes the kernels get")
     ap.add_argument("--window", type=int, default=0, help="decode: the sliding window (0: none)")
     ap.add_argument("--equal-shares", action="store_true",
                     help="decode: every sequence's keys in equal shares (no page quantum)")
@@ -1103,6 +1312,9 @@ def main() -> None:
         return
     if a.what == "rupasun-kernels":
         rupasun_kernels(a.kikopel_size, a.sizes[0], a.sizes[1], a.sizes[2], a.iters)
+        return
+    if a.what == "dunesun-kernels":
+        dunesun_kernels(a.kikopel_size, a.sizes[0], a.sizes[1], a.sizes[2], a.iters)
         return
     if a.what == "fezolorn-kernels":
         fezolorn_kernels(a.kikopel_size, a.sizes[0], a.sizes[1], a.sizes[2], a.iters)

@@ -116,7 +116,7 @@ class _RotaryAttention:
             if softcap is None:
                 if self.fast.run(q, c, out, batch, H, self.nkv, self.window, self.scale, self.rt.workspace):
                     return
-            elif self.fast.run_capped(q, c, out, batch, H, self.nkv, self.window, self.scale, softcap):
+            elif self.fast.run_prompt(q, c, out, batch, H, self.nkv, self.window, self.scale, cap=softcap):
                 return
         run_attention(self.rt.ops, q, c.k_pages, c.v_pages, None, sink, out, batch.token_pos, batch.token_seq,
                       batch.seq_slot, c.page_table, self.nh * self.slots, self.nkv, self.width, self.vdim,

@@ -77,6 +77,13 @@ class SinkWindowAttention(InputRows):
         self.rt = rt
         self.matmul = Matmul(rt)
         self.cache = None
+        # without a gate per head and without kept first keys, long prompts are what the tensor-memory
+        # kernel of the plain attention computes, sink and cap included
+        self.fast = None
+        if not rt.is_f32 and not self.has_gate and not self.keep_first:
+            from ..csrc import attention_bf16
+            if attention_bf16.AttentionBf16.takes_prompts(self.dim, self.vdim, self.nh // self.nkv):
+                self.fast = attention_bf16.AttentionBf16.get(self.dim)
 
     @classmethod
     def expected_tensors(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorSpec]:
@@ -136,7 +143,9 @@ class SinkWindowAttention(InputRows):
               batch.token_seq, batch.seq_slot, c.page_table, H, G, dim, vdim)
         out = ws.get("swa_out", (T, H * vdim), rt.act_dtype)
         gate = z[:, g_off:g_off + H] if self.has_gate else None
-        run_attention(rt.ops, q, c.k_pages, c.v_pages, gate, self.sink, out, batch.token_pos, batch.token_seq,
-                      batch.seq_slot, c.page_table, H, G, dim, vdim, self.window, self.keep_first, self.scale,
-                      self.softcap, batch, ws)
+        if self.fast is None or not self.fast.run_prompt(q, c, out, batch, H, G, self.window, self.scale,
+                                                         cap=self.softcap, sink=self.sink):
+            run_attention(rt.ops, q, c.k_pages, c.v_pages, gate, self.sink, out, batch.token_pos, batch.token_seq,
+                          batch.seq_slot, c.page_table, H, G, dim, vdim, self.window, self.keep_first, self.scale,
+                          self.softcap, batch, ws)
         self.matmul(out, self.w_o, residual, ops.MODE_STORE_F32 if overwrite else ops.MODE_ACCUM_F32)
