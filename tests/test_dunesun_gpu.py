@@ -284,3 +284,209 @@ def test_replay_program_and_command_line(tmp_path):
         for tok in line.split():
             assert int(tok) == int(np.argmax(plain.forward(cfg, w, seq)[-1]))
             seq.append(int(tok))
+
+
+# ---------------------------------------------------------------------------------------------
+# Kernels alone
+# ---------------------------------------------------------------------------------------------
+def _ops(dtype):
+    from torchless_rs_b200.csrc import ops
+    return ops.core_ops(dtype)
+
+
+def _dev(a, dtype=torch.float32):
+    return torch.as_tensor(np.asarray(a), dtype=dtype).cuda().contiguous()
+
+
+def _i32(a):
+    return torch.as_tensor(np.asarray(a, dtype=np.int32)).cuda()
+
+
+def _np(t):
+    return t.detach().double().cpu().numpy()
+
+
+def _pieces(n, cuts):
+    """(start, count) of the steps that feed n tokens in pieces of `cuts`, the rest one by one."""
+    out, at = [], 0
+    for c in list(cuts) + [1] * n:
+        if at >= n:
+            break
+        c = min(c, n - at)
+        out.append((at, c))
+        at += c
+    return out
+
+
+# ---- convolution, step sizes, kept inputs -----------------------------------------------------------------
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 6, 16])
+def test_preparation_at_a_sequences_start_and_across_steps(taps, dtype):
+    """Two sequences in one step, in pieces of every size, in slots that held another sequence's inputs before
+    (cleared when the slot was taken, as the cache does): nothing looks past a sequence's start or at its neighbour."""
+    rng = np.random.default_rng(taps)
+    H, ch, n = 3, 150, 75
+    col_x, col_dt = 5, 5 + ch + 2
+    z = [rng.normal(size=(n, col_dt + H)) for _ in range(2)]
+    w, b = rng.normal(size=(ch, taps)), rng.normal(size=ch)
+    A, dtb = rng.normal(size=H), rng.normal(size=H) * 3
+    o, wd = _ops(dtype), _dev(w)
+    bd, na, dbd = _dev(b), _dev(-np.exp(A)), _dev(dtb)
+    want = [plain.silu(plain.short_convolution(x[:, col_x:col_x + ch], w, b)) for x in z]
+    for cuts in ([n], [1, 1, 1, 2, 2, 3, 16, 17], [16, 32, 2], [40]):
+        kept = torch.full((4, max(taps - 1, 1), ch), 7.0, device="cuda")
+        kept[2] = 0.0
+        kept[1] = 0.0
+        for at, c in _pieces(n, cuts):
+            c2 = c                                              # both sequences bring the same number
+            zz = _dev(np.concatenate([z[0][at:at + c], z[1][at:at + c2]]))
+            xbc = torch.empty((c + c2, ch), device="cuda", dtype=dtype)
+            dtla = torch.empty((c + c2, H, 2), device="cuda")
+            o.ssd_prep(zz, col_x, col_dt, wd, bd, kept, xbc, dtla, na, dbd, _i32([0, c, c + c2]), _i32([2, 1]))
+            tol = 1e-5 if dtype == torch.float32 else 8e-3
+            for k in (0, 1):
+                got = _np(xbc[k * c:k * c + c])
+                ref = want[k][at:at + c]
+                assert (np.abs(got - ref) <= tol * (1 + np.abs(ref))).all(), (cuts, at, c, k)
+                dt = plain.softplus(z[k][at:at + c, col_dt:] + dtb)
+                d = _np(dtla[k * c:k * c + c])
+                assert np.allclose(d[..., 0], dt, rtol=2e-6, atol=1e-7)
+                assert np.allclose(d[..., 1], -np.exp(A) * dt, rtol=4e-6, atol=1e-7)
+        if taps > 1:
+            assert np.allclose(_np(kept[2]), z[0][n - taps + 1:, col_x:col_x + ch], atol=1e-6)
+            assert np.allclose(_np(kept[1]), z[1][n - taps + 1:, col_x:col_x + ch], atol=1e-6)
+            assert (kept[0] == 7.0).all() and (kept[3] == 7.0).all(), "a slot that is not in the step was written"
+
+
+# ---- the recurrence -----------------------------------------------------------------------------------------
+SSD_SIZES = [(3, 3, 20, 12), (1, 1, 33, 5), (6, 2, 16, 16), (4, 2, 64, 32), (4, 1, 128, 80), (2, 1, 256, 64), (8, 2, 48, 48),
+             (2, 2, 300, 20)]
+
+
+def _ssd_case(rng, n, H, G, N, P, dtype, spread=True):
+    """(xbc, dt, A_log, D) with values that the activation type holds; decays from nearly none to nothing left
+    within a token, side by side in a head."""
+    xbc = torch.from_numpy(rng.normal(size=(n, H * P + 2 * G * N)) / 2).to(dtype)
+    dt = np.exp(rng.normal(-1.0, 1.2, (n, H)))
+    if spread:
+        dt[rng.random((n, H)) < 0.02] = 25.0            # the state is all but gone after such a token
+    A = rng.normal(-2.0, 1.0, H)
+    A[0] = 1.2
+    return xbc, dt.astype(np.float32), A.astype(np.float32), rng.normal(size=H).astype(np.float32)
+
+
+def _ssd_plain(xbc, dt, A, D, H, G, N, P, S0=None):
+    """y of the plain recurrence and the end state, from S0."""
+    n = xbc.shape[0]
+    v = _np(xbc)
+    x, B, C = v[:, :H * P].reshape(n, H, P), v[:, H * P:H * P + G * N].reshape(n, G, N), v[:, H * P + G * N:].reshape(n, G, N)
+    if S0 is None:
+        S0 = np.zeros((H, N, P))
+    y, S = np.zeros((n, H, P)), S0.copy()
+    la = (-np.exp(A.astype(np.float64)).astype(np.float32) * dt).astype(np.float64)
+    for t in range(n):
+        for h in range(H):
+            S[h] = np.exp(la[t, h]) * S[h] + float(dt[t, h]) * np.outer(B[t, h // (H // G)], x[t, h])
+            y[t, h] = S[h].T @ C[t, h // (H // G)] + float(D[h]) * x[t, h]
+    return y.reshape(n, H * P), S
+
+
+def _ssd_run(o, xbc, dt, A, D, state, starts, slots, H, G, chunked=None):
+    na = -np.exp(A.astype(np.float64)).astype(np.float32)
+    dtla = _dev(np.stack([dt, (na * dt).astype(np.float32)], axis=-1))
+    P = state.shape[3]
+    y = torch.full((xbc.shape[0], H * P), float("nan"), device="cuda")
+    o.ssd_scan(xbc.cuda(), dtla, _dev(D), state, y, _i32(starts), _i32(slots), H, G, chunked=chunked)
+    return _np(y)
+
+
+@pytest.mark.parametrize("H,G,N,P", SSD_SIZES)
+def test_recurrence_in_32_bit_and_short_steps(H, G, N, P):
+    """The walk: two sequences in used slots, in pieces; every piece goes on from the state the one before left."""
+    rng = np.random.default_rng(N + P)
+    for dtype in (torch.float32, torch.bfloat16):
+        o = _ops(dtype)
+        for cuts in ([20], [1, 2, 7, 8, 9], []):
+            n = 27
+            cases = [_ssd_case(rng, n, H, G, N, P, dtype) for _ in range(2)]
+            A, D = cases[0][2], cases[0][3]
+            state = torch.randn((5, H, N, P), device="cuda")
+            state[3] = 0.0
+            S1 = _np(state[0])
+            got = [[], []]
+            for at, c in _pieces(n, cuts):
+                xbc = torch.cat([k[0][at:at + c] for k in cases])
+                y = _ssd_run(o, xbc, np.concatenate([k[1][at:at + c] for k in cases]), A, D, state, [0, c, 2 * c], [3, 0], H, G,
+                             chunked=False)
+                got[0].append(y[:c])
+                got[1].append(y[c:])
+            for k, S0 in ((0, None), (1, S1)):
+                ref, S = _ssd_plain(cases[k][0], cases[k][1], A, D, H, G, N, P, S0)
+                scale = np.abs(ref).max()
+                assert np.abs(np.concatenate(got[k]) - ref).max() <= 4e-6 * scale, (dtype, cuts, k)
+                assert np.abs(_np(state[3 if k == 0 else 0]) - S).max() <= 4e-6 * max(1.0, np.abs(S).max())
+
+
+@pytest.mark.parametrize("H,G,N,P", [s for s in SSD_SIZES if s[2] % 16 == 0 and s[3] % 16 == 0])
+def test_recurrence_in_chunks(H, G, N, P):
+    """Chunks on the tensor cores against the plain recurrence on the same bfloat16 x, B and C: what the state, the
+    decays and the weights lose is held to 1e-4 of the largest output (bfloat16 state or weights would lose 4e-3),
+    also where strong decays stand beside weak ones.  Lengths at and around a chunk, unequal sequences, used slots."""
+    rng = np.random.default_rng(N * P)
+    o = _ops(torch.bfloat16)
+    for lens in ([128], [129, 1, 127], [64, 300], [2, 255, 256]):
+        cases = [_ssd_case(rng, n, H, G, N, P, torch.bfloat16) for n in lens]
+        A, D = cases[0][2], cases[0][3]
+        state = torch.randn((len(lens) + 2, H, N, P), device="cuda")
+        slots = [len(lens) + 1 - i for i in range(len(lens))]
+        S0 = [_np(state[s]) for s in slots]
+        other = state[0].clone()
+        starts = np.concatenate([[0], np.cumsum(lens)])
+        y = _ssd_run(o, torch.cat([c[0] for c in cases]), np.concatenate([c[1] for c in cases]), A, D, state, starts, slots, H,
+                     G, chunked=True)
+        assert np.isfinite(y).all()
+        for i, c in enumerate(cases):
+            ref, S = _ssd_plain(c[0], c[1], A, D, H, G, N, P, S0[i])
+            err = np.abs(y[starts[i]:starts[i + 1]] - ref).max()
+            assert err <= 1e-4 * np.abs(ref).max(), f"lengths {lens}, sequence {i}: {err:.2e} of {np.abs(ref).max():.1f}"
+            assert np.abs(_np(state[slots[i]]) - S).max() <= 5e-5 * max(1.0, np.abs(S).max())
+        assert torch.equal(state[0], other), "a slot that is not in the step was written"
+
+
+@pytest.mark.parametrize("chunked", [False, True])
+def test_a_value_written_far_back_is_recalled(chunked):
+    """One token writes a value with a key of its own, 700 tokens of other keys and hardly any decay later it is
+    read; after a token that decays everything it is gone."""
+    H, G, N, P, n = 2, 1, 32, 16, 720
+    o = _ops(torch.bfloat16)
+    x, B, C = np.zeros((n, H, P)), np.zeros((n, G, N)), np.zeros((n, G, N))
+    rng = np.random.default_rng(3)
+    B[:, :, 1:] = rng.choice([-1.0, 1.0], (n, G, N - 1)) * 0.5
+    x[:] = rng.choice([-1.0, 1.0], (n, H, P))
+    B[9] = 0.0
+    B[9, 0, 0] = 2.0                                   # entry 0 is written by token 9 alone
+    x[9] = 4.0
+    C[709:, 0, 0] = 1.0                                 # and read by tokens 709 on
+    dt = np.full((n, H), 0.25, dtype=np.float32)
+    dt[715, :] = 1e5                                    # everything before is gone
+    A = np.full(H, np.log(1e-3), dtype=np.float32)
+    x[715] = 0.0
+    xbc = torch.from_numpy(np.concatenate([x.reshape(n, -1), B.reshape(n, -1), C.reshape(n, -1)], axis=1)).to(torch.bfloat16)
+    state = torch.zeros((1, H, N, P), device="cuda")
+    y = _ssd_run(o, xbc, dt, A, np.zeros(H, dtype=np.float32), state, [0, n], [0], H, G, chunked=chunked).reshape(n, H, P)
+    assert np.allclose(y[709], 0.25 * 2.0 * 4.0 * np.exp(-1e-3 * 0.25 * 700), rtol=1e-4)
+    assert np.abs(y[:9]).max() == 0.0 and np.abs(y[715:]).max() < 1e-30
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("inner,parts", [(36, 1), (36, 3), (30, 6), (256, 2), (4096, 1), (4096, 8), (20000, 1)])
+def test_gate_then_norm_in_parts(inner, parts, dtype):
+    rng = np.random.default_rng(inner)
+    T = 5
+    y, z, w = rng.normal(size=(T, inner)) * 3, rng.normal(size=(T, inner + 12)) * 2, rng.normal(size=inner)
+    y[:, :inner // parts] *= 50.0                       # parts of very different size: each by its own root mean square
+    out = torch.empty((T, inner), device="cuda", dtype=dtype)
+    _ops(dtype).ssd_gate_norm(_dev(y), _dev(z)[:, :inner], _dev(w), 1e-5, out, parts)
+    ref = plain.gated_group_norm(y, z[:, :inner], w, parts, 1e-5)
+    tol = 1e-5 if dtype == torch.float32 else 8e-3
+    assert (np.abs(_np(out) - ref) <= tol * (0.1 + np.abs(ref))).all()
