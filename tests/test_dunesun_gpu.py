@@ -490,3 +490,279 @@ def test_gate_then_norm_in_parts(inner, parts, dtype):
     ref = plain.gated_group_norm(y, z[:, :inner], w, parts, 1e-5)
     tol = 1e-5 if dtype == torch.float32 else 8e-3
     assert (np.abs(_np(out) - ref) <= tol * (0.1 + np.abs(ref))).all()
+
+
+# ---- query and key norms over the whole projection, cache pages ------------------------------------------------
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,dim,vdim", [(4, 2, 16, 16), (3, 3, 10, 7), (1, 1, 13, 40), (8, 2, 64, 48), (40, 8, 128, 128)])
+def test_norm_over_the_whole_projection_and_cache_write(H, G, dim, vdim, dtype):
+    rng = np.random.default_rng(dim)
+    PAGE = 64
+    for lens, past in (([1, 1, 1], [0, 63, 64]), ([70, 3], [62, 5])):
+        T = sum(lens)
+        z = rng.normal(size=(T, (H + G) * dim + G * vdim + 8))
+        z[:, :dim] *= 20.0                              # one head dominates: a norm per head would show
+        qw, kw = rng.normal(size=H * dim), rng.normal(size=G * dim)
+        B, per_seq = len(lens), 3
+        table = rng.permutation(B * per_seq + 2)[:B * per_seq].reshape(B, per_seq)
+        kp = torch.full((B * per_seq + 2, G, PAGE, dim), 9.0, device="cuda", dtype=dtype)
+        vp = torch.full((B * per_seq + 2, G, vdim, PAGE), 9.0, device="cuda", dtype=dtype)
+        pos = np.concatenate([np.arange(p, p + n) for p, n in zip(past, lens)])
+        seq = np.repeat(np.arange(B), lens)
+        slot = np.arange(B)[::-1].copy()
+        q = torch.empty((T, H * dim), device="cuda", dtype=dtype)
+        tab = np.zeros((B, per_seq), dtype=np.int32)
+        tab[slot] = table
+        _ops(dtype).qk_whole_norm_cache_write(_dev(z), None, _dev(qw), _dev(kw), 1e-6, q, kp, vp, _i32(pos), _i32(seq), _i32(slot),
+                                              _i32(tab), H, G, dim, vdim)
+        rq = plain.rms_normalise(z[:, :H * dim], 1e-6) * qw
+        rk = plain.rms_normalise(z[:, H * dim:(H + G) * dim], 1e-6) * kw
+        rv = z[:, (H + G) * dim:(H + G) * dim + G * vdim]
+        tol = 1e-5 if dtype == torch.float32 else 8e-3
+        assert (np.abs(_np(q) - rq) <= tol * (0.01 + np.abs(rq))).all()
+        written = torch.zeros_like(kp[:, 0, :, 0], dtype=torch.bool)
+        for t in range(T):
+            page, at = table[seq[t], pos[t] // PAGE], pos[t] % PAGE
+            written[page, at] = True
+            k, v = _np(kp[page, :, at]).reshape(-1), _np(vp[page, :, :, at]).reshape(-1)
+            assert (np.abs(k - rk[t]) <= tol * (0.01 + np.abs(rk[t]))).all() and (np.abs(v - rv[t]) <= tol * (0.01 + np.abs(rv[t]))).all()
+        assert (kp.permute(0, 2, 1, 3)[~written] == 9.0).all() and (vp.permute(0, 3, 1, 2)[~written] == 9.0).all()
+
+
+# ---- attention: window edges, far keys, one added to the denominator ----------------------------------------------
+class _View:
+    def __init__(self, kp, vp, table):
+        self.k_pages, self.v_pages, self.page_table = kp, vp, table
+
+
+class _Step:
+    def __init__(self, start, lens, slot, max_new, n, is_decode):
+        self.seq_start, self.seq_len, self.seq_slot, self.max_new, self.n_seqs, self.is_decode = start, lens, slot, max_new, n, is_decode
+        self.max_len = None
+
+
+def _attend(dtype, q, kp, vp, table, first, n, H, G, dim, vdim, window, scale, sink, tensor_memory):
+    """The queries of positions first .. first + n - 1 of one sequence, by the kernel the step would take."""
+    from torchless_rs_b200.csrc.attention_bf16 import AttentionBf16
+    from torchless_rs_b200.parts.sink_attention import run_attention
+    pos = _i32(np.arange(first, first + n))
+    seq, slot, start, lens = _i32([0] * n), _i32([0]), _i32([0, n]), _i32([first + n])
+    out = torch.full((n, H * vdim), float("nan"), device="cuda", dtype=dtype)
+    step = _Step(start, lens, slot, n, 1, n == 1)
+    if tensor_memory:
+        assert AttentionBf16.get(dim).run_prompt(q, _View(kp, vp, table), out, step, H, G, window, scale, sink=sink)
+    else:
+        run_attention(_ops(dtype), q, kp, vp, None, sink, out, pos, seq, slot, table, H, G, dim, vdim, window, 0, scale, None,
+                      step)
+    return _np(out).reshape(n, H, vdim)
+
+
+@pytest.mark.parametrize("dtype,H,G,dim,vdim", [(torch.float32, 4, 2, 24, 20), (torch.float32, 2, 1, 64, 300),
+                                                (torch.bfloat16, 4, 2, 24, 20), (torch.bfloat16, 4, 4, 32, 48),
+                                                (torch.bfloat16, 8, 2, 64, 64), (torch.bfloat16, 4, 1, 128, 128),
+                                                (torch.bfloat16, 2, 1, 200, 400)])
+@pytest.mark.parametrize("window", [None, 1, 20, 64, 65, 130])
+def test_keys_that_stand_out_at_a_windows_edge_and_far_back(dtype, H, G, dim, vdim, window):
+    """A key scaled so that its score stands out by tens: just inside the window it decides the output, just outside
+    it changes nothing; keys on page borders and hundreds of tokens back; as a decode step, a few tokens and a
+    long run (the tensor-memory kernel where it takes the sizes)."""
+    from torchless_rs_b200.csrc.attention_bf16 import AttentionBf16
+    rng = np.random.default_rng(dim + (window or 0))
+    n, PAGE = 330, 64
+    scale = 1.0 / np.sqrt(dim)
+    k = rng.normal(size=(n, G, dim)) * 0.3
+    v = rng.normal(size=(n, G, vdim))
+    q = rng.normal(size=(n, H, dim)) * 0.3
+    u = np.ones(dim) / np.sqrt(dim)                     # the direction of the pairs that stand out
+    loud = [0, 63, 64, 127, 190, 300]
+    for j in loud:
+        k[j] += 6.0 * np.sqrt(dim) * u * (1 if j % 2 else 0.8)
+    q += 1.0 * np.sqrt(dim) ** 0.5 * u
+    pages = (n + PAGE - 1) // PAGE
+    table = rng.permutation(pages + 1)[:pages]
+    kp = torch.zeros((pages + 1, G, PAGE, dim), device="cuda", dtype=dtype)
+    vp = torch.zeros((pages + 1, G, vdim, PAGE), device="cuda", dtype=dtype)
+    kd, vd, qd = _dev(k, dtype), _dev(v, dtype), _dev(q, dtype)
+    for p in range(pages):
+        m = min(PAGE, n - p * PAGE)
+        kp[table[p], :, :m] = kd[p * PAGE:p * PAGE + m].permute(1, 0, 2)
+        vp[table[p], :, :, :m] = vd[p * PAGE:p * PAGE + m].permute(1, 2, 0)
+    tab = _i32(table[None])
+    # the oracle on the values the kernel gets
+    qs, ks, vs = _np(qd), _np(kd), _np(vd)
+    mask = plain.visible(n, window)
+    ref = np.zeros((n, H, vdim))
+    for h in range(H):
+        ref[:, h] = plain.softmax_plus_one(qs[:, h] @ ks[:, h // (H // G)].T * scale, mask) @ vs[:, h // (H // G)]
+    sink = torch.zeros(H, device="cuda")
+    tol = 2e-5 if dtype == torch.float32 else 1.2e-2
+    edges = sorted({min(n - 1, j + d) for j in loud for d in ((window or 1) - 1, window or 1)})
+    takes = dtype == torch.bfloat16 and AttentionBf16.takes_prompts(dim, vdim, H // G)
+    runs = [(e, 1, False) for e in edges] + [(60, 5, False), (125, 7, False), (0, n, False)]
+    if takes:
+        runs += [(0, n, True), (64, n - 64, True), (101, 200, True)]
+    for first, m, tm in runs:
+        got = _attend(dtype, qd[first:first + m].reshape(m, -1).contiguous(), kp, vp, tab, first, m, H, G, dim, vdim, window, scale,
+                      sink, tm)
+        r = ref[first:first + m]
+        assert np.isfinite(got).all()
+        bad = np.abs(got - r) > tol * (1.0 + np.abs(r))
+        assert not bad.any(), (f"window {window}, queries {first}..{first + m - 1}, tensor memory {tm}: "
+                               f"{np.abs(got - r).max():.2e} at {np.argwhere(bad)[0]}")
+
+
+@pytest.mark.parametrize("dim", [48, 64, 128])
+@pytest.mark.parametrize("level", [-40.0, -3.0, 0.0, 3.0, 40.0])
+def test_the_added_one_takes_its_share(dim, level):
+    """Every score equals `level`: a key's weight is e^level / (1 + n e^level), nearly nothing far below zero, 1 / n far
+    above; by every kernel and however many tokens the step brings."""
+    from torchless_rs_b200.csrc.attention_bf16 import AttentionBf16
+    H, G, n = 4, 2, 200
+    k = torch.zeros((4, G, 64, dim), device="cuda", dtype=torch.bfloat16)
+    k[:, :, :, 0] = 1.0
+    v = torch.ones((4, G, dim, 64), device="cuda", dtype=torch.bfloat16)
+    q = torch.zeros((n, H, dim), device="cuda", dtype=torch.bfloat16)
+    q[:, :, 0] = level
+    tab = _i32([[2, 0, 3, 1]])
+    sink = torch.zeros(H, device="cuda")
+    seen = np.minimum(np.arange(n) + 1, 90)
+    want = 1.0 / (1.0 + np.exp(-level) / seen)
+    for first, m, tm in ((0, n, False), (150, 1, False), (7, 3, False)) + (((0, n, True),) if dim % 64 == 0 else ()):
+        got = _attend(torch.bfloat16, q[first:first + m].reshape(m, -1).contiguous(), k, v, tab, first, m, H, G, dim, dim, 90, 1.0,
+                      sink, tm)
+        assert np.allclose(got, want[first:first + m, None, None], rtol=1e-2), (first, m, tm)
+
+
+# ---- experts and the closing kernel -----------------------------------------------------------------------------
+@pytest.mark.parametrize("E,top", [(1, 1), (3, 3), (5, 2), (33, 4), (64, 8), (512, 6)])
+def test_choice_by_logits_and_softmax_over_the_chosen(E, top):
+    rng = np.random.default_rng(E)
+    T = 70
+    z, b = rng.normal(size=(T, E + 3)) * 2, rng.normal(size=E) * 2
+    z[0], b0 = 0.0, np.zeros(E)                        # all tie: the lower indices
+    z[1, :E] = -1e30                                    # far below zero, still a softmax over the chosen
+    for bias in (b.astype(np.float32), b0.astype(np.float32), None):
+        zz = z.astype(np.float32)
+        idx = torch.empty((T, top), dtype=torch.int32, device="cuda")
+        wt = torch.empty((T, top), device="cuda")
+        _ops(torch.float32).moe_route_chosen(_dev(zz)[:, :E], None if bias is None else _dev(bias), top, idx, wt)
+        zb = zz[:, :E] + (0 if bias is None else bias)
+        ri, rw = plain.route(zb.astype(np.float64), top)
+        assert (idx.cpu().numpy() == ri).all()
+        assert np.allclose(_np(wt), rw, rtol=2e-6, atol=1e-7)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("W,ff,E,top,T", [(96, 40, 6, 2, 50), (82, 33, 3, 2, 7), (256, 128, 8, 3, 200), (128, 64, 4, 4, 1)])
+def test_experts_products_and_closing_kernel(W, ff, E, top, T, dtype):
+    """Plan, grouped products with silu(gate) * up, and the closing kernel with every combination of its terms,
+    against the plain experts; one expert is chosen by nobody, one by every token."""
+    rng = np.random.default_rng(W + T)
+    o = _ops(dtype)
+    rnd = lambda *s: _np(torch.from_numpy(rng.normal(size=s)).to(dtype))
+    h, wg, wu, wd = rnd(T, W), rnd(E, ff, W) / W ** 0.5, rnd(E, ff, W) / W ** 0.5, rnd(E, W, ff) / ff ** 0.5
+    cast = lambda a: _np(torch.from_numpy(a).to(dtype))
+    wg, wu, wd = cast(wg), cast(wu), cast(wd)
+    z = rng.normal(size=(T, E))
+    if top < E:
+        z[:, 1] = -50.0
+    z[:, 0] = 50.0
+    ri, rw = plain.route(z, top)
+    idx, wt = _i32(ri), _dev(rw)
+    off = torch.empty(E + 1, dtype=torch.int32, device="cuda")
+    row_token = torch.empty(T * top, dtype=torch.int32, device="cuda")
+    row_of = torch.empty((T, top), dtype=torch.int32, device="cuda")
+    o.moe_plan(idx, E, off, row_token, row_of)
+    act = torch.empty((T * top, ff), device="cuda", dtype=dtype)
+    yk = torch.empty((T * top, W), device="cuda")
+    w_up = _dev(np.concatenate([wg, wu], axis=1), dtype)
+    o.moe_gemm(_dev(h, dtype), row_token, w_up, act, off, up=True, act=0)
+    o.moe_gemm(act, None, _dev(wd, dtype), yk, off, up=False)
+    want = np.zeros((T, W))
+    for e in range(E):
+        r, k = np.nonzero(ri == e)
+        want[r] += rw[r, k][:, None] * ((plain.silu(h[r] @ wg[e].T) * (h[r] @ wu[e].T)) @ wd[e].T)
+    x, ys, sg = rng.normal(size=(T, W)), rng.normal(size=(T, W)), rng.normal(size=(T, 5)) * 2
+    rows, vec, w = rng.normal(size=(T, W)), rng.normal(size=W), rng.normal(size=W)
+    tol = 2e-5 if dtype == torch.float32 else 1.5e-2
+    for use in range(32):
+        xd = _dev(x)
+        ref = x.copy()
+        kw = {}
+        if use & 1:
+            kw["experts"], ref = (yk, row_of, wt), ref + want
+        if use & 2:
+            kw["shared"], ref = (_dev(ys), _dev(sg)[:, 3] if use & 16 else None), ref + (plain.sigmoid(sg[:, 3:4]) if use & 16 else 1.0) * ys
+        if use & 4:
+            kw["add_rows"], ref = _dev(rows), ref + rows
+        if use & 8:
+            kw["add_vec"], ref = _dev(vec), ref + vec
+        xn = torch.empty((T, W), device="cuda", dtype=dtype)
+        if use % 3:
+            kw.update(w_next=_dev(w), eps_next=1e-3, xn=xn)
+        o.close_block(xd, **kw)
+        assert np.abs(_np(xd) - ref).max() <= tol * 4, use
+        if use % 3:
+            assert (np.abs(_np(xn) - plain.rms_normalise(ref, 1e-3) * w) <= tol * 4).all(), use
+
+
+@pytest.mark.parametrize("W,T", [(4096, 3), (4096, 600), (20000, 2), (20003, 2)])
+def test_closing_kernel_on_wide_rows(W, T):
+    rng = np.random.default_rng(W)
+    x, rows, vec, w = rng.normal(size=(T, W)), rng.normal(size=(T, W)), rng.normal(size=W), rng.normal(size=W)
+    xd, xn = _dev(x), torch.empty((T, W), device="cuda")
+    _ops(torch.float32).close_block(xd, None, None, _dev(rows), _dev(vec), _dev(w), 1e-6, xn)
+    ref = x + rows + vec
+    assert np.allclose(_np(xd), ref, atol=1e-5) and np.allclose(_np(xn), plain.rms_normalise(ref, 1e-6) * w, atol=2e-5)
+
+
+def test_embedding_keeps_a_copy_and_adds_the_first_passs_row():
+    rng = np.random.default_rng(0)
+    V, W, P, T = 30, 37, 16, 9
+    tab, pos, vec = rng.normal(size=(V, W)), rng.normal(size=(P, W)), rng.normal(size=W)
+    tok, at = rng.integers(0, V, T), rng.integers(0, P, T)
+    x, copy = torch.empty((T, W), device="cuda"), torch.empty((T, W), device="cuda")
+    o = _ops(torch.float32)
+    for with_pos in (True, False):
+        o.embed(_i32(tok), _dev(tab), x, scale=0.5, position_table=_dev(pos) if with_pos else None, token_pos=_i32(at), copy=copy,
+                add_vec=_dev(vec))
+        ref = 0.5 * tab[tok] + (pos[at] if with_pos else 0.0)
+        assert np.allclose(_np(copy), ref, atol=1e-6) and np.allclose(_np(x), ref + vec, atol=1e-6)
+
+
+def test_blocks_that_take_no_addend_work_in_repeated_passes():
+    """A pre-norm model whose layers run twice, with what stands before a pass added by a kernel of its own: the
+    block before must not have prepared its successor's norm from the stream without it."""
+    import dataclasses
+    from helpers_gpu import TinyModel
+    from tiny import CONFIGS as MISTRAL
+    from torchless_rs_b200.config import PassStart
+    from torchless_rs_b200.engine.engine import Engine
+    tm = TinyModel("A", "float32", seed=3, max_tokens=256)
+    spec = tm.engine.spec
+    n = len(spec.layers)
+    W = spec.hidden_size
+    rng = np.random.default_rng(2)
+    toks = [int(t) for t in rng.integers(0, MISTRAL["A"]["vocab_size"], 20)]
+    new = dataclasses.replace(spec, order=tuple(range(n)) * 2, pass_table_name="steps", pass_rows=2,
+                              pass_starts={0: PassStart(0), n: PassStart(1, True)})
+    w = {k: torch.from_numpy(np.asarray(v, dtype=np.float32)) for k, v in tm.weights.items()}
+    w["steps"] = torch.from_numpy(rng.normal(size=(2, W)).astype(np.float32))
+    eng = Engine(new, w, tm.engine.rt, 256, use_graphs=False)
+    added = []
+    ops = eng.rt.ops
+    real = ops.close_block
+    def spy(x, *a, **k):
+        before = x.clone()
+        real(x, *a, **k)
+        added.append((x - before).cpu().numpy())
+    ops.close_block = spy
+    try:
+        s = eng.start_sequences(1)
+        whole = eng.step(s, [toks], "all").cpu().numpy().copy()
+    finally:
+        del ops.close_block
+    assert len(added) == 1 and np.allclose(added[0], _np(w[spec.embedding_name])[toks] + _np(w["steps"])[1], atol=1e-5)
+    s2 = eng.start_sequences(1)
+    one = np.concatenate([eng.step(s2, [[t]], "last").cpu().numpy().copy() for t in toks])
+    assert np.allclose(whole, one, atol=2e-4 * np.abs(whole).max())

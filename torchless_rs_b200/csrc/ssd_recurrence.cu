@@ -795,7 +795,7 @@ extern "C" int tl_ssd_chunked(const void* xbc, const float* dtla, const float* D
   const size_t NS = N + SSD_PAD, PS = SSD_PT + SSD_PAD;
   const size_t sm1 = (SSD_Q * NS + 2 * SSD_Q * PS) * 2;
   const size_t one = (2 * SSD_Q * NS + (SSD_Q + 2 * (size_t)N) * PS) * 2, more = (SSD_Q + 2 * (size_t)N) * PS * 2;
-  const size_t most = 220 * 1024;       // and some 3 KB that are not dynamic
+  const size_t most = 223 * 1024;       // and some 3 KB that are not dynamic
   if (one > most) return TL_ERR_UNSUPPORTED;
   static bool set = false;
   if (!set) {
