@@ -69,6 +69,8 @@ def _register_builtin() -> None:
     register_architecture("Fezolorn")(FezolornConfig)
     from .dunesun import DunesunConfig
     register_architecture("Dunesun")(DunesunConfig)
+    from .beralix import BeralixConfig
+    register_architecture("Beralix")(BeralixConfig)
 
 
 _register_builtin()

@@ -17,8 +17,9 @@
 // Per token, from the 32-bit down-projections:
 //   cq[t, :]  = dq[t, :] / rms * wq                          (query latent, activation type)
 //   page row  = [ dkv[t, :rank] / rms * wc | rotate(dkv[t, rank:rank+rot]) ]   at the token's place
+// Without a query latent (q_rank = 0) only the page row is written.
 // Rotation: entry i of the rot part pairs with entry i + dims/2 (i < dims/2), angle =
-// position * inv_freq[i]; entries from `dims` on pass unchanged.
+// position * inv_freq[i], sine and cosine times `amp`; entries from `dims` on pass unchanged.
 // ---------------------------------------------------------------------------
 __global__ void latent_prep_kernel(const float* __restrict__ dq, int ld_dq, const float* __restrict__ dkv,
                                    int ld_dkv, const float* __restrict__ wq, const float* __restrict__ wc,
@@ -26,7 +27,7 @@ __global__ void latent_prep_kernel(const float* __restrict__ dq, int ld_dq, cons
                                    const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                                    const int* __restrict__ seq_slot, const int* __restrict__ page_table,
                                    int table_stride, const float* __restrict__ inv_freq, int q_rank, int rank,
-                                   int rot, int dims) {
+                                   int rot, int dims, float amp) {
   __shared__ float scratch[33];
   pdl_wait();
   pdl_launch_dependents();
@@ -36,9 +37,9 @@ __global__ void latent_prep_kernel(const float* __restrict__ dq, int ld_dq, cons
   float sq = 0.0f, sc = 0.0f;
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x) sq = fmaf(a[i], a[i], sq);
   for (int i = threadIdx.x; i < rank; i += blockDim.x) sc = fmaf(b[i], b[i], sc);
-  sq = block_sum(sq, scratch);
+  if (q_rank > 0) sq = block_sum(sq, scratch);
   sc = block_sum(sc, scratch);
-  const float rq = sqrtf(sq / (float)q_rank + eps), rc = sqrtf(sc / (float)rank + eps);
+  const float rq = q_rank > 0 ? sqrtf(sq / (float)q_rank + eps) : 1.0f, rc = sqrtf(sc / (float)rank + eps);
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
     cq[(size_t)t * q_rank + i] = from_f32<act_t>((a[i] / rq) * wq[i]);
   const int pos = token_pos[t];
@@ -51,6 +52,8 @@ __global__ void latent_prep_kernel(const float* __restrict__ dq, int ld_dq, cons
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn, cs;
     sincosf((float)pos * inv_freq[i], &sn, &cs);
+    sn *= amp;
+    cs *= amp;
     const float u = r[i], v = r[i + half];
     row[rank + i] = from_f32<act_t>(u * cs - v * sn);
     row[rank + i + half] = from_f32<act_t>(v * cs + u * sn);
@@ -62,31 +65,37 @@ extern "C" int TL_NAME(tl_latent_prep)(const float* dq, int ld_dq, const float* 
                                        const float* wc, float eps, void* cq, void* pages, const int* token_pos,
                                        const int* token_seq, const int* seq_slot, const int* page_table,
                                        int table_stride, const float* inv_freq, int T, int q_rank, int rank,
-                                       int rot, int dims, cudaStream_t stream) {
+                                       int rot, int dims, float amp, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (q_rank <= 0 || rank <= 0 || rot < 0 || dims < 0 || dims > rot || (dims & 1)) return TL_ERR_BAD_ARG;
+  if (q_rank < 0 || rank <= 0 || rot < 0 || dims < 0 || dims > rot || (dims & 1)) return TL_ERR_BAD_ARG;
   return tl_launch(latent_prep_kernel, dim3(T), dim3(128), 0, stream, dq, ld_dq, dkv, ld_dkv, wq, wc, eps,
                    (act_t*)cq, (act_t*)pages, token_pos, token_seq, seq_slot, page_table, table_stride, inv_freq,
-                   q_rank, rank, rot, dims);
+                   q_rank, rank, rot, dims, amp);
 }
 
 // ---------------------------------------------------------------------------
 // One small product per head:  C[t, h, n] = sum_k A[t, h, k] * W[h, n, k]
 //   A 32-bit, row stride lda, head h at column h * a_head;  W [heads, N, K] in the activation type;
 //   C row stride ldc, head h at column h * c_head.
-// epilogue 0: C 32-bit = product;  1: C (activation type) = product * sigmoid(G[t, h * N + n]),
-// G 32-bit with row stride ldg (an output gate), or the product alone where G is null.
+// epilogue 0: C 32-bit = product;  1: C (activation type) = product * sigmoid(g), or the product alone where G
+// is null.  G: 32-bit with row stride ldg; an output gate per entry (g_one 0: g = G[t, h * N + n]) or per head
+// (g_one 1: g = G[t, h]).
 // 64 x 64 tiles, 16 K-elements a step, 256 threads with 4 x 4 outputs each; 32-bit FFMA.
 // ---------------------------------------------------------------------------
 #define HW_BM 64
 #define HW_BN 64
 #define HW_BK 16
 
+__device__ __forceinline__ float hw_gate(const float* G, int ldg, int g_one, int m, int h, int n, int N) {
+  const float x = G[(size_t)m * ldg + (g_one ? (size_t)h : (size_t)h * N + n)];
+  return 1.0f / (1.0f + expf(-x));
+}
+
 template <int EPI>
 __global__ void __launch_bounds__(256)
 headwise_gemm_kernel(const float* __restrict__ A, int lda, int a_head, const act_t* __restrict__ W,
-                     void* __restrict__ C, int ldc, int c_head, const float* __restrict__ G, int ldg, int M,
-                     int N, int K) {
+                     void* __restrict__ C, int ldc, int c_head, const float* __restrict__ G, int ldg,
+                     int g_one, int M, int N, int K) {
   __shared__ float As[HW_BK][HW_BM + 4];
   __shared__ float Ws[HW_BK][HW_BN + 4];
   pdl_wait();
@@ -133,7 +142,7 @@ headwise_gemm_kernel(const float* __restrict__ A, int lda, int a_head, const act
       if (EPI == 0) {
         ((float*)C)[at] = acc[i][j];
       } else {
-        const float g = G != nullptr ? 1.0f / (1.0f + expf(-G[(size_t)m * ldg + (size_t)h * N + n])) : 1.0f;
+        const float g = G != nullptr ? hw_gate(G, ldg, g_one, m, h, n, N) : 1.0f;
         ((act_t*)C)[at] = from_f32<act_t>(acc[i][j] * g);
       }
     }
@@ -144,8 +153,8 @@ headwise_gemm_kernel(const float* __restrict__ A, int lda, int a_head, const act
 template <int EPI>
 __global__ void __launch_bounds__(256)
 headwise_gemv_kernel(const float* __restrict__ A, int lda, int a_head, const act_t* __restrict__ W,
-                     void* __restrict__ C, int ldc, int c_head, const float* __restrict__ G, int ldg, int M,
-                     int N, int K) {
+                     void* __restrict__ C, int ldc, int c_head, const float* __restrict__ G, int ldg,
+                     int g_one, int M, int N, int K) {
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31;
@@ -162,15 +171,15 @@ headwise_gemv_kernel(const float* __restrict__ A, int lda, int a_head, const act
     if (EPI == 0) {
       ((float*)C)[at] = acc;
     } else {
-      const float g = G != nullptr ? 1.0f / (1.0f + expf(-G[(size_t)m * ldg + (size_t)h * N + n])) : 1.0f;
+      const float g = G != nullptr ? hw_gate(G, ldg, g_one, m, h, n, N) : 1.0f;
       ((act_t*)C)[at] = from_f32<act_t>(acc * g);
     }
   }
 }
 
 extern "C" int TL_NAME(tl_headwise_gemm)(const float* A, int lda, int a_head, const void* W, void* C, int ldc,
-                                         int c_head, const float* G, int ldg, int M, int N, int K, int heads,
-                                         int epilogue, cudaStream_t stream) {
+                                         int c_head, const float* G, int ldg, int g_one, int M, int N, int K,
+                                         int heads, int epilogue, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || heads <= 0) return 0;
   if (K <= 0 || epilogue < 0 || epilogue > 1) return TL_ERR_BAD_ARG;
   if (heads > 65535) return TL_ERR_UNSUPPORTED;
@@ -178,17 +187,17 @@ extern "C" int TL_NAME(tl_headwise_gemm)(const float* A, int lda, int a_head, co
     dim3 grid((N + 7) / 8, M, heads);
     if (epilogue == 0)
       return tl_launch(headwise_gemv_kernel<0>, grid, dim3(256), 0, stream, A, lda, a_head, (const act_t*)W, C,
-                       ldc, c_head, G, ldg, M, N, K);
+                       ldc, c_head, G, ldg, g_one, M, N, K);
     return tl_launch(headwise_gemv_kernel<1>, grid, dim3(256), 0, stream, A, lda, a_head, (const act_t*)W, C, ldc,
-                     c_head, G, ldg, M, N, K);
+                     c_head, G, ldg, g_one, M, N, K);
   }
   dim3 grid((N + HW_BN - 1) / HW_BN, (M + HW_BM - 1) / HW_BM, heads);
   if (grid.y > 65535) return TL_ERR_UNSUPPORTED;
   if (epilogue == 0)
     return tl_launch(headwise_gemm_kernel<0>, grid, dim3(256), 0, stream, A, lda, a_head, (const act_t*)W, C, ldc,
-                     c_head, G, ldg, M, N, K);
+                     c_head, G, ldg, g_one, M, N, K);
   return tl_launch(headwise_gemm_kernel<1>, grid, dim3(256), 0, stream, A, lda, a_head, (const act_t*)W, C, ldc,
-                   c_head, G, ldg, M, N, K);
+                   c_head, G, ldg, g_one, M, N, K);
 }
 
 // ---------------------------------------------------------------------------
@@ -229,7 +238,8 @@ latent_attn_kernel(const float* __restrict__ qa, int ld_qa, int qa_head, const f
                    const act_t* __restrict__ pages, float* __restrict__ o, const int* __restrict__ token_pos,
                    const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                    const int* __restrict__ page_table, int table_stride, const float* __restrict__ inv_freq,
-                   const float* __restrict__ sink, int heads, int rank, int rot, int dims, int window, float scale) {
+                   const float* __restrict__ sink, int heads, int rank, int rot, int dims, int window, float scale,
+                   float amp) {
   extern __shared__ float qs[];          // [rank + rot]
   __shared__ float ps[LAT_THREADS];
   __shared__ int pg[LAT_THREADS];
@@ -249,6 +259,8 @@ latent_attn_kernel(const float* __restrict__ qa, int ld_qa, int qa_head, const f
     for (int i = tid; i < half; i += LAT_THREADS) {
       float sn, cs;
       sincosf((float)pos * inv_freq[i], &sn, &cs);
+      sn *= amp;
+      cs *= amp;
       const float u = r[i], v = r[i + half];
       qs[rank + i] = (u * cs - v * sn) * scale;
       qs[rank + i + half] = (v * cs + u * sn) * scale;
@@ -320,14 +332,15 @@ extern "C" int TL_NAME(tl_latent_attn)(const float* qa, int ld_qa, int qa_head, 
                                        const void* pages, float* o, const int* token_pos, const int* token_seq,
                                        const int* seq_slot, const int* page_table, int table_stride,
                                        const float* inv_freq, const float* sink, int T, int heads, int rank,
-                                       int rot, int dims, int window, float scale, cudaStream_t stream) {
+                                       int rot, int dims, int window, float scale, float amp,
+                                       cudaStream_t stream) {
   if (T <= 0) return 0;
   if (heads <= 0 || rank <= 0 || rot < 0 || dims > rot || (dims & 1)) return TL_ERR_BAD_ARG;
   if (rank > LAT_THREADS * LAT_MAX_PER_THREAD || heads > 65535 || (rank + rot) * sizeof(float) > 40 * 1024)
     return TL_ERR_UNSUPPORTED;
   return tl_launch(latent_attn_kernel, dim3(T, heads), dim3(LAT_THREADS), (size_t)(rank + rot) * sizeof(float),
                    stream, qa, ld_qa, qa_head, q, ldq, q_head, q_off, (const act_t*)pages, o, token_pos, token_seq, seq_slot,
-                   page_table, table_stride, inv_freq, sink, heads, rank, rot, dims, window, scale);
+                   page_table, table_stride, inv_freq, sink, heads, rank, rot, dims, window, scale, amp);
 }
 
 #if TL_DTYPE == 1
@@ -391,7 +404,7 @@ latent_attn_mma_kernel(const float* __restrict__ qa, int ld_qa, int qa_head, con
                        const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                        const int* __restrict__ page_table, int table_stride, const float* __restrict__ inv_freq,
                        const float* __restrict__ sink, int T, int heads, int rank, int rot, int dims, int window,
-                       float scale, int splits) {
+                       float scale, float amp, int splits) {
   extern __shared__ __align__(16) unsigned char lm_smem[];
   const int width = rank + rot, pitch = width + 8;
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(lm_smem);          // [TB][16][pitch]
@@ -424,7 +437,7 @@ latent_attn_mma_kernel(const float* __restrict__ qa, int ld_qa, int qa_head, con
     for (int i = tl; i < half; i += LM_THREADS) {
       float sn, cs;
       sincosf((float)pos * inv_freq[i], &sn, &cs);
-      cs_s[i] = make_float2(cs, sn);
+      cs_s[i] = make_float2(cs * amp, sn * amp);
     }
     __syncthreads();
     const float qscale = scale * 1.4426950408889634f;      // log2(e): the softmax below works in base 2
@@ -723,8 +736,8 @@ extern "C" int tl_latent_attn_mma(const float* qa, int ld_qa, int qa_head, const
                                   int q_off, const void* pages, float* o, float* part, const int* token_pos,
                                   const int* token_seq, const int* seq_slot, const int* page_table,
                                   int table_stride, const float* inv_freq, const float* sink, int T, int heads,
-                                  int rank, int rot, int dims, int window, float scale, int splits,
-                                  cudaStream_t stream) {
+                                  int rank, int rot, int dims, int window, float scale, float amp,
+                                  int splits, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (rank % 16 || rot % 16 || rank > 512 || rank <= 0 || dims > rot || (dims & 1) || rot > 1024 || splits < 1 ||
       (splits > 1 && part == nullptr))
@@ -749,7 +762,7 @@ extern "C" int tl_latent_attn_mma(const float* qa, int ld_qa, int qa_head, const
     rc = tl_launch(latent_attn_mma_kernel<NTP, TBV>, grid, dim3(LM_THREADS * TBV), smem, stream, qa, ld_qa,  \
                    qa_head, q, ldq, q_head, q_off, (const __nv_bfloat16*)pages, o, part, token_pos, token_seq, \
                    seq_slot, page_table, table_stride, inv_freq, sink, T, heads, rank, rot, dims, window,    \
-                   scale, splits);                                                                                  \
+                   scale, amp, splits);                                                                             \
   }
 #define LM_LAUNCH(NTP) \
   { if (many) LM_LAUNCH_TB(NTP, 4) else LM_LAUNCH_TB(NTP, 1) }
@@ -765,9 +778,10 @@ extern "C" int tl_latent_attn_mma(const float* qa, int ld_qa, int qa_head, const
 }
 
 // ---------------------------------------------------------------------------
-// The per-head value up-projection with the output gate on tensor cores (bfloat16 build), for steps of
-// many tokens:  C[t, h, n] = sigmoid(G[t, h N + n]) * sum_k A[t, h, k] W[h, n, k],  A 32-bit (rounded to
-// bfloat16 on its way into shared memory), W and C bfloat16.  A block computes 64 rows x 64 outputs of
+// The per-head products on tensor cores (bfloat16 build), for steps of many tokens:
+//   C[t, h, n] = gate * sum_k A[t, h, k] W[h, n, k],  A 32-bit (rounded to bfloat16 on its way into shared
+// memory), W bfloat16; C bfloat16, with the output gate of the kernels above if there is one (the value
+// up-projection), or 32-bit without a gate (OUT32: queries on their way into the latent space).  A block computes 64 rows x 64 outputs of
 // one head; each of its four warps 16 rows; K goes in steps of 32 through shared memory.
 // ---------------------------------------------------------------------------
 #define HM_BM 64
@@ -775,10 +789,11 @@ extern "C" int tl_latent_attn_mma(const float* qa, int ld_qa, int qa_head, const
 #define HM_BK 32
 #define HM_PITCH (HM_BK + 8)
 
+template <bool OUT32>
 __global__ void __launch_bounds__(128)
 headwise_mma_kernel(const float* __restrict__ A, int lda, int a_head, const __nv_bfloat16* __restrict__ W,
-                    __nv_bfloat16* __restrict__ C, int ldc, int c_head, const float* __restrict__ G, int ldg,
-                    int M, int N, int K) {
+                    void* __restrict__ C, int ldc, int c_head, const float* __restrict__ G, int ldg,
+                    int g_one, int M, int N, int K) {
   __shared__ __align__(16) __nv_bfloat16 As[HM_BM * HM_PITCH];
   __shared__ __align__(16) __nv_bfloat16 Ws[HM_BN * HM_PITCH];
   pdl_wait();
@@ -839,26 +854,36 @@ headwise_mma_kernel(const float* __restrict__ A, int lda, int a_head, const __nv
       const int n = n0 + nt * 8 + qd * 2;
       if (n >= N) continue;          // N is even (checked by the launcher), so n + 1 < N too
       float v0 = acc[nt][2 * r], v1 = acc[nt][2 * r + 1];
-      if (G != nullptr) {
+      const size_t at = (size_t)m * ldc + (size_t)h * c_head + n;
+      if (OUT32) {
+        *reinterpret_cast<float2*>((float*)C + at) = make_float2(v0, v1);
+        continue;
+      }
+      if (G != nullptr && g_one) {
+        const float gt = hw_gate(G, ldg, 1, m, h, n, N);
+        v0 *= gt;
+        v1 *= gt;
+      } else if (G != nullptr) {
         const float2 gt = *reinterpret_cast<const float2*>(G + (size_t)m * ldg + (size_t)h * N + n);
         v0 *= 1.0f / (1.0f + expf(-gt.x));
         v1 *= 1.0f / (1.0f + expf(-gt.y));
       }
-      *reinterpret_cast<uint32_t*>(C + (size_t)m * ldc + (size_t)h * c_head + n) = pack_bf16(v0, v1);
+      *reinterpret_cast<uint32_t*>((__nv_bfloat16*)C + at) = pack_bf16(v0, v1);
     }
   }
 }
 
 // Returns TL_ERR_UNSUPPORTED for sizes or alignments it does not take (the FFMA kernel then runs).
 extern "C" int tl_headwise_mma(const float* A, int lda, int a_head, const void* W, void* C, int ldc, int c_head,
-                               const float* G, int ldg, int M, int N, int K, int heads, cudaStream_t stream) {
+                               const float* G, int ldg, int g_one, int M, int N, int K, int heads, int out32,
+                               cudaStream_t stream) {
   if (M <= 0 || N <= 0 || heads <= 0) return 0;
-  if (K % 8 || N % 2 || lda % 4 || a_head % 4 || ldc % 2 || c_head % 2 || ldg % 2 ||
-      ((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((uintptr_t)C & 3) || ((uintptr_t)G & 7) || heads > 65535 ||
+  if (K % 8 || N % 2 || lda % 4 || a_head % 4 || ldc % 2 || c_head % 2 || (!g_one && (ldg % 2 || ((uintptr_t)G & 7))) ||
+      ((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((uintptr_t)C & (out32 ? 7 : 3)) || heads > 65535 ||
       (M + HM_BM - 1) / HM_BM > 65535)
     return TL_ERR_UNSUPPORTED;
   dim3 grid((N + HM_BN - 1) / HM_BN, (M + HM_BM - 1) / HM_BM, heads);
-  return tl_launch(headwise_mma_kernel, grid, dim3(128), 0, stream, A, lda, a_head, (const __nv_bfloat16*)W,
-                   (__nv_bfloat16*)C, ldc, c_head, G, ldg, M, N, K);
+  return tl_launch(out32 ? headwise_mma_kernel<true> : headwise_mma_kernel<false>, grid, dim3(128), 0, stream, A, lda,
+                   a_head, (const __nv_bfloat16*)W, C, ldc, c_head, G, ldg, g_one, M, N, K);
 }
 #endif

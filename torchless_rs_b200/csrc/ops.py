@@ -142,7 +142,8 @@ class CoreOps:
                      "tl_rotary_cache_write", "tl_diff_heads", "tl_sigmoid_gate", "tl_norm_add_norm", "tl_relu_squared",
                      "tl_clamped_glu", "tl_delta_prep", "tl_conv_state_update", "tl_delta_scan", "tl_silu_rows",
                      "tl_weighted_sum", "tl_close_block", "tl_moe_route_chosen", "tl_qk_whole_norm_cache_write",
-                     "tl_ssd_prep", "tl_ssd_walk", "tl_ssd_gate_norm"):
+                     "tl_ssd_prep", "tl_ssd_walk", "tl_ssd_gate_norm", "tl_layernorm",
+                     "tl_layernorm_add_layernorm", "tl_selective_scan"):
             fn = getattr(self.lib, f"{base}_{self.suffix}")
             fn.restype = c_int
             setattr(self, "_" + base, fn)
@@ -367,39 +368,48 @@ class CoreOps:
                                   c_int(F), _stream()), "poly_norm")
 
     # ---- attention through latents ----------------------------------------------------------------
-    def latent_prep(self, dq: torch.Tensor, dkv: torch.Tensor, wq: torch.Tensor, wc: torch.Tensor, eps: float,
-                    cq: torch.Tensor, pages: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
+    def latent_prep(self, dq: Optional[torch.Tensor], dkv: torch.Tensor, wq: Optional[torch.Tensor], wc: torch.Tensor,
+                    eps: float, cq: Optional[torch.Tensor], pages: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
                     seq_slot: torch.Tensor, page_table: torch.Tensor, inv_freq: Optional[torch.Tensor],
-                    rank: int, rot: int, dims: int) -> None:
-        """cq = norm(dq) * wq; the token's page row = [norm(dkv[:, :rank]) * wc | rotate(dkv[:, rank:])]."""
+                    rank: int, rot: int, dims: int, amplitude: float = 1.0) -> None:
+        """cq = norm(dq) * wq (none of the three: no query latent); the token's page row =
+        [norm(dkv[:, :rank]) * wc | rotate(dkv[:, rank:])], sine and cosine times `amplitude`."""
         for t, n in ((dq, "query down-projection"), (dkv, "key/value down-projection")):
+            if t is None and dq is None:
+                continue
             _need(t, torch.float32, n, contiguous=False)
             if t.stride(1) != 1:
                 raise KernelError(f"latent_prep: {n} must have contiguous rows")
-        _need(wq, torch.float32, "query latent norm weight")
+        if (dq is None) != (cq is None) or (dq is None) != (wq is None):
+            raise KernelError("latent_prep: a query latent needs its projection, weight and output")
+        if dq is not None:
+            _need(wq, torch.float32, "query latent norm weight")
+            _need(cq, self.act_dtype, "query latent")
         _need(wc, torch.float32, "latent norm weight")
-        _need(cq, self.act_dtype, "query latent")
         _need(pages, self.act_dtype, "latent pages")
         _need(page_table, torch.int32, "page table")
-        T, q_rank = cq.shape
-        if dq.shape != (T, q_rank) or dkv.shape != (T, rank + rot) or wq.numel() != q_rank or \
-                wc.numel() != rank or pages.shape[1:] != (PAGE, rank + rot):
+        T, q_rank = dkv.shape[0], 0
+        if dq is not None:
+            q_rank = cq.shape[1]
+            if dq.shape != (T, q_rank) or cq.shape[0] != T or wq.numel() != q_rank:
+                raise KernelError("latent_prep: sizes do not match")
+        if dkv.shape != (T, rank + rot) or wc.numel() != rank or pages.shape[1:] != (PAGE, rank + rot):
             raise KernelError("latent_prep: sizes do not match")
         if dims:
             _need(inv_freq, torch.float32, "inv_freq")
             if inv_freq.numel() != dims // 2:
                 raise KernelError("latent_prep: inv_freq must have dims/2 entries")
         _check(self._tl_latent_prep(
-            _ptr(dq), c_int(dq.stride(0)), _ptr(dkv), c_int(dkv.stride(0)), _ptr(wq), _ptr(wc), c_float(eps),
+            _ptr(dq), c_int(dq.stride(0) if dq is not None else 0), _ptr(dkv), c_int(dkv.stride(0)), _ptr(wq), _ptr(wc), c_float(eps),
             _ptr(cq), _ptr(pages), _ptr(token_pos), _ptr(token_seq), _ptr(seq_slot), _ptr(page_table),
             c_int(page_table.stride(0)), _ptr(inv_freq if dims else None), c_int(T), c_int(q_rank), c_int(rank),
-            c_int(rot), c_int(dims), _stream()), "latent_prep")
+            c_int(rot), c_int(dims), c_float(amplitude), _stream()), "latent_prep")
 
     def headwise_gemm(self, a: torch.Tensor, a_head: int, w: torch.Tensor, c: torch.Tensor, c_head: int,
                       gate: Optional[torch.Tensor] = None, act_out: bool = False) -> None:
         """c[t, h * c_head + n] = sum_k a[t, h * a_head + k] * w[h, n, k] for every head h; with `gate`
-        ([T, heads * N] 32-bit) the result is multiplied by sigmoid(gate) and `c` is of the activation
-        type; without a gate `c` is 32-bit, or, with `act_out`, of the activation type."""
+        ([T, heads * N] 32-bit, or [T, heads]: one per head) the result is multiplied by sigmoid(gate) and `c` is of
+        the activation type; without a gate `c` is 32-bit, or, with `act_out`, of the activation type."""
         act_out = act_out or gate is not None
         _need(a, torch.float32, "headwise a", contiguous=False)
         _need(w, self.act_dtype, "headwise w")
@@ -409,31 +419,34 @@ class CoreOps:
         if a.stride(1) != 1 or c.stride(1) != 1 or c.shape[0] != M or \
                 a.shape[1] < (heads - 1) * a_head + K or c.shape[1] < (heads - 1) * c_head + N:
             raise KernelError("headwise_gemm: sizes do not match")
-        ldg = 0
+        ldg = per_head = 0
         if gate is not None:
             _need(gate, torch.float32, "headwise gate", contiguous=False)
-            if gate.shape != (M, heads * N) or gate.stride(1) != 1:
-                raise KernelError("headwise_gemm: the gate must be [rows, heads * outputs]")
-            ldg = gate.stride(0)
-        if act_out and M > 16 and self.act_dtype == torch.bfloat16:
+            if gate.shape not in ((M, heads * N), (M, heads)) or gate.stride(1) != 1:
+                raise KernelError("headwise_gemm: the gate must be [rows, heads * outputs] or [rows, heads]")
+            ldg, per_head = gate.stride(0), int(gate.shape[1] == heads)
+        if M > 16 and self.act_dtype == torch.bfloat16:
             # many rows: the tensor-core kernel, where sizes and alignments allow it
             self.lib.tl_headwise_mma.restype = c_int
             st = self.lib.tl_headwise_mma(_ptr(a), c_int(a.stride(0)), c_int(a_head), _ptr(w), _ptr(c),
-                                          c_int(c.stride(0)), c_int(c_head), _ptr(gate), c_int(ldg), c_int(M),
-                                          c_int(N), c_int(K), c_int(heads), _stream())
+                                          c_int(c.stride(0)), c_int(c_head), _ptr(gate), c_int(ldg),
+                                          c_int(per_head), c_int(M), c_int(N), c_int(K), c_int(heads),
+                                          c_int(0 if act_out else 1), _stream())
             if st != -2:
                 _check(st, "headwise_mma")
                 return
         _check(self._tl_headwise_gemm(_ptr(a), c_int(a.stride(0)), c_int(a_head), _ptr(w), _ptr(c),
-                                      c_int(c.stride(0)), c_int(c_head), _ptr(gate), c_int(ldg), c_int(M), c_int(N),
-                                      c_int(K), c_int(heads), c_int(1 if act_out else 0), _stream()),
+                                      c_int(c.stride(0)), c_int(c_head), _ptr(gate), c_int(ldg),
+                                      c_int(per_head), c_int(M), c_int(N), c_int(K), c_int(heads),
+                                      c_int(1 if act_out else 0), _stream()),
                "headwise_gemm")
 
     def latent_attn(self, qa: torch.Tensor, qa_head: int, q: torch.Tensor, q_head: int, q_off: int,
                     pages: torch.Tensor, out: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
                     seq_slot: torch.Tensor, page_table: torch.Tensor, inv_freq: Optional[torch.Tensor], heads: int,
                     rank: int, rot: int, dims: int, window: Optional[int], scale: float,
-                    max_keys: Optional[int] = None, workspace=None, sink: Optional[torch.Tensor] = None) -> None:
+                    max_keys: Optional[int] = None, workspace=None, sink: Optional[torch.Tensor] = None,
+                    amplitude: float = 1.0) -> None:
         """out[t, h, :] = softmax over the visible positions of ((qa[t, h] . c + rotate(q_rot[t, h]) . r) *
         scale) times the positions' c; page rows are [c | r].  Head h's latent-space query starts at column
         h * qa_head of `qa`, its part to rotate at column h * q_head + q_off of `q` (one buffer may be both).
@@ -441,7 +454,8 @@ class CoreOps:
         In bfloat16 the tensor-core kernel runs where the sizes allow it (rank and rot multiples of 16,
         rank <= 512); `max_keys` (an upper bound of the keys a token of the step sees) lets it cut the keys
         of a step of few tokens into parts, whose partial sums lie in a buffer of `workspace`.  `sink` (one
-        32-bit number per head) adds exp(sink[h]) to the softmax's denominator, once."""
+        32-bit number per head) adds exp(sink[h]) to the softmax's denominator, once.  The rotation's sine and cosine
+        are multiplied by `amplitude`."""
         if sink is not None:
             _need(sink, torch.float32, "sink")
             if sink.numel() != heads:
@@ -473,7 +487,7 @@ class CoreOps:
                     c_int(q_off), _ptr(pages), _ptr(out), _ptr(part), _ptr(token_pos), _ptr(token_seq),
                     _ptr(seq_slot), _ptr(page_table), c_int(page_table.stride(0)), _ptr(inv_freq if dims else None),
                     _ptr(sink), c_int(T), c_int(heads), c_int(rank), c_int(rot), c_int(dims), c_int(window or 0),
-                    c_float(scale), c_int(splits), _stream()), "latent_attn_mma")
+                    c_float(scale), c_float(amplitude), c_int(splits), _stream()), "latent_attn_mma")
                 if splits > 1:
                     _check(0, "latent_attn_merge")
                 return
@@ -481,7 +495,8 @@ class CoreOps:
             _ptr(qa), c_int(qa.stride(0)), c_int(qa_head), _ptr(q), c_int(q.stride(0)), c_int(q_head), c_int(q_off),
             _ptr(pages), _ptr(out), _ptr(token_pos), _ptr(token_seq), _ptr(seq_slot), _ptr(page_table),
             c_int(page_table.stride(0)), _ptr(inv_freq if dims else None), _ptr(sink), c_int(T), c_int(heads),
-            c_int(rank), c_int(rot), c_int(dims), c_int(window or 0), c_float(scale), _stream()), "latent_attn")
+            c_int(rank), c_int(rot), c_int(dims), c_int(window or 0), c_float(scale), c_float(amplitude), _stream()),
+            "latent_attn")
 
     # ---- gated linear recurrence ------------------------------------------------------------------
     def gated_scan(self, z: torch.Tensor, bias: torch.Tensor, low: torch.Tensor, state: torch.Tensor,
@@ -815,7 +830,8 @@ class CoreOps:
                            v_pages: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
                            seq_slot: torch.Tensor, page_table: torch.Tensor, nq: int, nk: int, nv: int, dim: int,
                            vdim: int, slots: int = 1, bias: Optional[torch.Tensor] = None,
-                           values_are_keys: bool = False) -> None:
+                           values_are_keys: bool = False, amplitude: float = 1.0,
+                           first_values: Optional[torch.Tensor] = None, mix: Optional[float] = None) -> None:
         """The projections `z` (32-bit rows: `nq` query vectors and `nk` key vectors of `dim`, then `nv` value
         heads of `vdim`): the first `rot` entries of every query and key vector are rotated by the token's
         position (`style` 0: pairs (i, i + rot/2), 1: pairs (2i, 2i + 1)), then, with `unit_norm`, the vector
@@ -823,7 +839,9 @@ class CoreOps:
         key row of the pages holds `slots` key vectors side by side and query vector j becomes a row of that
         width that is zero outside slot j % slots.  `bias` (32-bit, one number per column of `z`) is added as
         the columns are read.  With `values_are_keys` `z` holds no value columns: a value head is the key
-        vector of its head as projected (bias included), before rotation and norm."""
+        vector of its head as projected (bias included), before rotation and norm.  The rotation's sine and cosine
+        are multiplied by `amplitude`.  `first_values` ([T, nv * vdim] 32-bit) receives the values, or, with `mix`
+        (a number), holds an earlier layer's: the values written are then (1 - mix) v + mix first_values."""
         _need(z, torch.float32, "projections", contiguous=False)
         _need(q_out, self.act_dtype, "q out")
         _need(k_pages, self.act_dtype, "k pages")
@@ -846,12 +864,19 @@ class CoreOps:
             _need(inv_freq, torch.float32, "inverse frequencies")
             if inv_freq.numel() != rot // 2:
                 raise KernelError("rotary_cache_write: one inverse frequency per rotated pair is needed")
+        if first_values is not None:
+            _need(first_values, torch.float32, "an earlier layer's values")
+            if first_values.shape != (T, nv * vdim):
+                raise KernelError("rotary_cache_write: one row of values per token is needed for mixing")
+        elif mix is not None:
+            raise KernelError("rotary_cache_write: there are no values to mix with")
         _check(self._tl_rotary_cache_write(
             _ptr(z), c_int(z.stride(0)), _ptr(bias), c_int(v_col), _ptr(inv_freq if rot else None), c_int(rot),
             c_int(style),
             c_int(1 if unit_norm else 0), c_float(eps), _ptr(q_out), _ptr(k_pages), _ptr(v_pages), _ptr(token_pos),
             _ptr(token_seq), _ptr(seq_slot), _ptr(page_table), c_int(page_table.stride(0)), c_int(T), c_int(nq),
-            c_int(nk), c_int(nv), c_int(dim), c_int(vdim), c_int(slots), _stream()), "rotary_cache_write")
+            c_int(nk), c_int(nv), c_int(dim), c_int(vdim), c_int(slots), c_float(amplitude), _ptr(first_values),
+            c_int(0 if mix is None else 1), c_float(mix or 0.0), _stream()), "rotary_cache_write")
 
     def diff_heads(self, a: torch.Tensor, lam: float, eps: float, mult: float, out: torch.Tensor, heads: int,
                    vdim: int) -> None:
@@ -1154,6 +1179,88 @@ class CoreOps:
             raise KernelError("ssd_gate_norm: sizes do not match")
         _check(self._tl_ssd_gate_norm(_ptr(y), _ptr(z), c_int(z.stride(0)), _ptr(w), c_float(eps), _ptr(out), c_int(T),
                                       c_int(inner), c_int(parts), _stream()), "ssd_gate_norm")
+
+    # ---- layer norms, and the selective scan with a decay per channel and state entry ---------------------
+    def layernorm(self, x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor,
+                  rows: Optional[torch.Tensor] = None) -> None:
+        """out = (x - mean) / sqrt(variance + eps) * weight + bias, row by row; `rows` (int32) picks rows of x."""
+        for t, n in ((x, "layernorm in"), (weight, "layernorm weight"), (bias, "layernorm bias")):
+            _need(t, torch.float32, n)
+        _need(out, self.act_dtype, "layernorm out")
+        n_rows, H = out.shape
+        if weight.numel() != H or bias.numel() != H or x.shape[1] != H or (rows is None and x.shape[0] != n_rows):
+            raise KernelError("layernorm: sizes do not match")
+        if rows is not None:
+            _need(rows, torch.int32, "layernorm rows")
+            if rows.numel() != n_rows:
+                raise KernelError("layernorm: one row index per output row is needed")
+        _check(self._tl_layernorm(_ptr(x), _ptr(rows), _ptr(weight), _ptr(bias), c_float(eps), _ptr(out), c_int(n_rows),
+                                  c_int(H), _stream()), "layernorm")
+
+    def layernorm_add_layernorm(self, y: torch.Tensor, w_out: torch.Tensor, b_out: torch.Tensor, eps_out: float,
+                                x: torch.Tensor, w_next: Optional[torch.Tensor] = None,
+                                b_next: Optional[torch.Tensor] = None, eps_next: float = 0.0,
+                                xn: Optional[torch.Tensor] = None) -> None:
+        """x += N(y) with weight and bias `w_out`, `b_out` (32-bit stream, in place); with `w_next`, also xn =
+        N_next(x) in the activation type."""
+        _need(y, torch.float32, "sublayer output", contiguous=False)
+        _need(x, torch.float32, "stream")
+        T, H = x.shape
+        if y.shape != (T, H) or y.stride(1) != 1:
+            raise KernelError("layernorm_add_layernorm: sizes do not match")
+        for t in (w_out, b_out) + ((w_next, b_next) if w_next is not None else ()):
+            _need(t, torch.float32, "layer norm weight or bias")
+            if t.numel() != H:
+                raise KernelError("layernorm_add_layernorm: sizes do not match")
+        if w_next is not None:
+            if xn is None or xn.shape != (T, H):
+                raise KernelError("layernorm_add_layernorm: the next norm needs a place for its result")
+            _need(xn, self.act_dtype, "normed stream")
+        _check(self._tl_layernorm_add_layernorm(
+            _ptr(y), c_int(y.stride(0)), _ptr(w_out), _ptr(b_out), c_float(eps_out), _ptr(x), _ptr(w_next), _ptr(b_next),
+            c_float(eps_next), _ptr(xn), c_int(T), c_int(H), _stream()), "layernorm_add_layernorm")
+
+    def conv_silu(self, z: torch.Tensor, col: int, taps_w: torch.Tensor, bias: torch.Tensor, kept: torch.Tensor,
+                  out: torch.Tensor, seq_start: torch.Tensor, seq_slot: torch.Tensor) -> None:
+        """out [T, channels] = silu(conv(z[:, col:]) + bias), the convolution and its kept inputs as in `ssd_prep`
+        (whose kernel this is, without step sizes)."""
+        _need(z, torch.float32, "projections", contiguous=False)
+        _need(out, self.act_dtype, "convolved channels")
+        for t, n in ((taps_w, "convolution taps"), (bias, "convolution bias"), (kept, "kept convolution inputs")):
+            _need(t, torch.float32, n)
+        T, channels = out.shape
+        taps = taps_w.shape[1]
+        if z.stride(1) != 1 or z.shape[0] != T or z.shape[1] < col + channels or taps_w.shape != (channels, taps) or \
+                bias.numel() != channels or kept.shape[2] != channels or kept.shape[1] != max(taps - 1, 1):
+            raise KernelError("conv_silu: sizes do not match")
+        _check(self._tl_ssd_prep(_ptr(z), c_int(z.stride(0)), c_int(col), c_int(0), _ptr(taps_w), _ptr(bias),
+                                 c_int(taps), _ptr(kept), _ptr(out), _ptr(None), _ptr(None), _ptr(None),
+                                 _ptr(seq_start), _ptr(seq_slot), c_int(T), c_int(seq_slot.numel()), c_int(channels),
+                                 c_int(0), _stream()), "conv_silu")
+
+    def selective_scan(self, x: torch.Tensor, zdt: torch.Tensor, dt_bias: torch.Tensor, bc: torch.Tensor, col_b: int,
+                       neg_a: torch.Tensor, D: torch.Tensor, z: torch.Tensor, state: torch.Tensor, y: torch.Tensor,
+                       seq_start: torch.Tensor, seq_slot: torch.Tensor) -> None:
+        """dt = softplus(zdt + dt_bias); S <- exp(dt neg_a) S + dt x B, y = (sum over the state of S C + D x) silu(z)
+        over each sequence's tokens of the step, from and into `state` [slots, channels, N]; B lies at column
+        `col_b` of `bc`, C behind it."""
+        _need(x, self.act_dtype, "scan input")
+        _need(bc, self.act_dtype, "scan B and C")
+        _need(y, self.act_dtype, "scan out")
+        for t, n in ((zdt, "step sizes"), (dt_bias, "step size bias"), (neg_a, "decay rates"), (D, "skip weights"),
+                     (state, "recurrent state")):
+            _need(t, torch.float32, n)
+        _need(z, torch.float32, "gate", contiguous=False)
+        T, channels = x.shape
+        N = neg_a.shape[1]
+        if zdt.shape != (T, channels) or dt_bias.numel() != channels or bc.shape[0] != T or bc.shape[1] < col_b + 2 * N or \
+                neg_a.shape[0] != channels or D.numel() != channels or z.shape != (T, channels) or z.stride(1) != 1 or \
+                state.shape[1:] != (channels, N) or y.shape != (T, channels):
+            raise KernelError("selective_scan: sizes do not match")
+        _check(self._tl_selective_scan(
+            _ptr(x), c_int(x.stride(0)), _ptr(zdt), _ptr(dt_bias), _ptr(bc), c_int(bc.stride(0)), c_int(col_b), _ptr(neg_a),
+            _ptr(D), _ptr(z), c_int(z.stride(0)), _ptr(state), _ptr(y), _ptr(seq_start), _ptr(seq_slot),
+            c_int(seq_slot.numel()), c_int(channels), c_int(N), _stream()), "selective_scan")
 
 
 class SamplingOps:

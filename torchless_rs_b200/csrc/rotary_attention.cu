@@ -7,13 +7,14 @@
 //                        k and plain v into the token's place in the pages.  `bias` (one number per
 //                        column of z, or null) is added as the columns are read; the value heads
 //                        start at column `v_col`, which may be where the key vectors start (the
-//                        values are then the keys as projected, before rotation and norm).
+//                        values are then the keys as projected, before rotation and norm).  Values may
+//                        be mixed with another layer's (ra_value below).
 //   diff_heads           o = a1 - lambda a2 per head, o / rms(o) * mult.
 //   sigmoid_gate         out *= sigmoid(gate), entry by entry.
 //
 // Rotation: the first `rot` entries of a vector turn in pairs by the angle pos * inv_freq[i],
 // pair i being (i, i + rot/2) (style 0) or (2i, 2i + 1) (style 1); the other entries pass.  Angle,
-// sine and cosine are 32-bit.
+// sine and cosine are 32-bit; sine and cosine are multiplied by `amp`.
 //
 // Several maps per head ("slots"): a key/value head's key row in the pages is its `slots` key
 // vectors side by side (slots * dim numbers), and query vector j is written as a row of the same
@@ -25,6 +26,22 @@
 #define RA_MAX_DIM 256
 #define RA_WARPS 4
 
+// What becomes of a token's value v on its way into the pages: with `first` ([tokens, nv * vdim] 32-bit) it is
+// left there for later layers (mix_in 0) or mixed with what an earlier layer left, (1 - lambda) v + lambda
+// first (mix_in 1).
+struct RaMix {
+  float* first;
+  int ld, mix_in;
+  float lambda;
+};
+__device__ __forceinline__ float ra_value(const RaMix& m, int t, int col, float v) {
+  if (m.first == nullptr) return v;
+  float* p = m.first + (size_t)t * m.ld + col;
+  if (m.mix_in) return (1.0f - m.lambda) * v + m.lambda * *p;
+  *p = v;
+  return v;
+}
+
 __global__ void __launch_bounds__(RA_WARPS * 32)
 rotary_cache_write_kernel(const float* __restrict__ z, int ldz, const float* __restrict__ bias, int v_col,
                           const float* __restrict__ inv_freq, int rot,
@@ -32,7 +49,8 @@ rotary_cache_write_kernel(const float* __restrict__ z, int ldz, const float* __r
                           act_t* __restrict__ k_pages, act_t* __restrict__ v_pages,
                           const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                           const int* __restrict__ seq_slot, const int* __restrict__ page_table,
-                          int table_stride, int nq, int nk, int nv, int dim, int vdim, int slots) {
+                          int table_stride, int nq, int nk, int nv, int dim, int vdim, int slots, float amp,
+                          RaMix mix) {
   __shared__ float vec[RA_WARPS][RA_MAX_DIM];
   pdl_wait();
   pdl_launch_dependents();
@@ -78,6 +96,8 @@ rotary_cache_write_kernel(const float* __restrict__ z, int ldz, const float* __r
             const float a = fpos * inv_freq[i];
             float sn, cs;
             sincosf(a, &sn, &cs);
+            sn *= amp;
+            cs *= amp;
             const float o = mine[partner];
             // (u, v) -> (u cos - v sin, v cos + u sin)
             v = first ? v * cs - o * sn : v * cs + o * sn;
@@ -112,7 +132,8 @@ rotary_cache_write_kernel(const float* __restrict__ z, int ldz, const float* __r
       const float* src = row + col;
       act_t* dst = v_pages + ((size_t)page * nv + g) * vdim * TL_PAGE + in_page;
       for (int d = lane; d < vdim; d += 32)
-        dst[(size_t)d * TL_PAGE] = from_f32<act_t>(src[d] + (bias != nullptr ? bias[col + d] : 0.0f));
+        dst[(size_t)d * TL_PAGE] =
+            from_f32<act_t>(ra_value(mix, t, g * vdim + d, src[d] + (bias != nullptr ? bias[col + d] : 0.0f)));
     }
   }
 }
@@ -166,7 +187,8 @@ rotary_cache_write_many_kernel(const float* __restrict__ z, int ldz, const float
                                act_t* __restrict__ k_pages, act_t* __restrict__ v_pages,
                                const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                                const int* __restrict__ seq_slot, const int* __restrict__ page_table,
-                               int table_stride, int T, int nq, int nk, int nv, int dim, int vdim, int slots) {
+                               int table_stride, int T, int nq, int nk, int nv, int dim, int vdim, int slots, float amp,
+                          RaMix mix) {
   extern __shared__ float ra_sm[];
   pdl_wait();
   pdl_launch_dependents();
@@ -180,7 +202,8 @@ rotary_cache_write_many_kernel(const float* __restrict__ z, int ldz, const float
     const float* src = z + col;
     for (int idx = threadIdx.x; idx < nt * vdim; idx += blockDim.x) {
       const int tt = idx / vdim, d = idx - tt * vdim;
-      ra_sm[tt * (vdim + 1) + d] = src[(size_t)(t0 + tt) * ldz + d] + (bias != nullptr ? bias[col + d] : 0.0f);
+      ra_sm[tt * (vdim + 1) + d] = ra_value(mix, t0 + tt, g * vdim + d,
+                                            src[(size_t)(t0 + tt) * ldz + d] + (bias != nullptr ? bias[col + d] : 0.0f));
     }
     __syncthreads();
     if (lane < nt) {
@@ -208,7 +231,7 @@ rotary_cache_write_many_kernel(const float* __restrict__ z, int ldz, const float
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn, c;
     sincosf(fpos * inv_freq[i], &sn, &c);
-    cs[i] = make_float2(c, sn);
+    cs[i] = make_float2(c * amp, sn * amp);
   }
   __syncthreads();
   float cur[R], nxt[R];
@@ -297,7 +320,8 @@ rotary_cache_write_vec_kernel(const float* __restrict__ z, int ldz, const float*
                               act_t* __restrict__ k_pages, act_t* __restrict__ v_pages,
                               const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                               const int* __restrict__ seq_slot, const int* __restrict__ page_table,
-                              int table_stride, int T, int nq, int nk, int nv, int vdim, int slots) {
+                              int table_stride, int T, int nq, int nk, int nv, int vdim, int slots, float amp,
+                          RaMix mix) {
   extern __shared__ float ra_sm[];
   pdl_wait();
   pdl_launch_dependents();
@@ -312,7 +336,8 @@ rotary_cache_write_vec_kernel(const float* __restrict__ z, int ldz, const float*
     const float* src = z + col;
     for (int idx = threadIdx.x; idx < nt * vdim; idx += blockDim.x) {
       const int tt = idx / vdim, d = idx - tt * vdim;
-      ra_sm[tt * (vdim + 1) + d] = src[(size_t)(t0 + tt) * ldz + d] + (bias != nullptr ? bias[col + d] : 0.0f);
+      ra_sm[tt * (vdim + 1) + d] = ra_value(mix, t0 + tt, g * vdim + d,
+                                            src[(size_t)(t0 + tt) * ldz + d] + (bias != nullptr ? bias[col + d] : 0.0f));
     }
     __syncthreads();
     if (lane < nt) {
@@ -339,7 +364,7 @@ rotary_cache_write_vec_kernel(const float* __restrict__ z, int ldz, const float*
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn, c;
     sincosf(fpos * inv_freq[i], &sn, &c);
-    cs[i] = make_float2(c, sn);
+    cs[i] = make_float2(c * amp, sn * amp);
   }
   const int slot = seq_slot[token_seq[t]];
   const int page = page_table[(size_t)slot * table_stride + pos / TL_PAGE];
@@ -403,8 +428,10 @@ extern "C" int TL_NAME(tl_rotary_cache_write)(const float* z, int ldz, const flo
                                               int unit_norm, float eps, void* q_out, void* k_pages, void* v_pages,
                                               const int* token_pos, const int* token_seq, const int* seq_slot,
                                               const int* page_table, int table_stride, int T, int nq, int nk,
-                                              int nv, int dim, int vdim, int slots, cudaStream_t stream) {
+                                              int nv, int dim, int vdim, int slots, float amp, float* first,
+                                              int mix_in, float lambda, cudaStream_t stream) {
   if (T <= 0) return 0;
+  const RaMix mix{first, nv * vdim, mix_in, lambda};
   if (nq < 1 || nk < 1 || nv < 1 || dim < 1 || vdim < 1 || slots < 1 || nq % slots || nk % slots ||
       nk / slots != nv || rot < 0 || rot > dim || (rot & 1) || (rot > 0 && inv_freq == nullptr) || v_col < 0)
     return TL_ERR_BAD_ARG;
@@ -422,7 +449,7 @@ extern "C" int TL_NAME(tl_rotary_cache_write)(const float* z, int ldz, const flo
 #define RA_VEC(LPV_)                                                                                                \
       return tl_launch(rotary_cache_write_vec_kernel<LPV_>, dim3(blocks), dim3(RAM_WARPS * 32), smem, stream, z,   \
                        ldz, bias, v_col, inv_freq, rot, style, unit_norm, eps, (act_t*)q_out, (act_t*)k_pages, (act_t*)v_pages, \
-                       token_pos, token_seq, seq_slot, page_table, table_stride, T, nq, nk, nv, vdim, slots)
+                       token_pos, token_seq, seq_slot, page_table, table_stride, T, nq, nk, nv, vdim, slots, amp, mix)
       if (dim == 16) RA_VEC(4);
       if (dim == 32) RA_VEC(8);
       if (dim == 64) RA_VEC(16);
@@ -432,7 +459,7 @@ extern "C" int TL_NAME(tl_rotary_cache_write)(const float* z, int ldz, const flo
 #define RA_MANY(R_)                                                                                                  \
     return tl_launch(rotary_cache_write_many_kernel<R_>, dim3(blocks), dim3(RAM_WARPS * 32), smem, stream, z, ldz,  \
                      bias, v_col, inv_freq, rot, style, unit_norm, eps, (act_t*)q_out, (act_t*)k_pages, (act_t*)v_pages,         \
-                     token_pos, token_seq, seq_slot, page_table, table_stride, T, nq, nk, nv, dim, vdim, slots)
+                     token_pos, token_seq, seq_slot, page_table, table_stride, T, nq, nk, nv, dim, vdim, slots, amp, mix)
     if (dim <= 32) RA_MANY(1);
     if (dim <= 64) RA_MANY(2);
     if (dim <= 128) RA_MANY(4);
@@ -442,7 +469,7 @@ extern "C" int TL_NAME(tl_rotary_cache_write)(const float* z, int ldz, const flo
   const dim3 grid(T, (vectors + RA_WARPS - 1) / RA_WARPS);
   return tl_launch(rotary_cache_write_kernel, grid, dim3(RA_WARPS * 32), 0, stream, z, ldz, bias, v_col, inv_freq, rot, style,
                    unit_norm, eps, (act_t*)q_out, (act_t*)k_pages, (act_t*)v_pages, token_pos, token_seq, seq_slot,
-                   page_table, table_stride, nq, nk, nv, dim, vdim, slots);
+                   page_table, table_stride, nq, nk, nv, dim, vdim, slots, amp, mix);
 }
 
 // a: [T][heads][2][vdim] (the two maps' outputs of every head); out: [T][heads][vdim].

@@ -126,7 +126,7 @@ extern "C" int TL_NAME(tl_ssd_prep)(const float* z, int ld, int col_x, int col_d
                                     const float* neg_a, const float* dt_bias, const int* seq_start,
                                     const int* seq_slot, int T, int B, int channels, int H, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
-  if (channels < 1 || H < 1 || taps < 1) return TL_ERR_BAD_ARG;
+  if (channels < 1 || H < 0 || taps < 1) return TL_ERR_BAD_ARG;     // H = 0: the convolution alone
   if (taps > SSD_MAX_TAPS) return TL_ERR_UNSUPPORTED;
   const int ch_blocks = (channels + 127) / 128;
   const int dt_blocks = (H * (T < SSD_STRIP ? T : SSD_STRIP) + 511) / 512;

@@ -6,6 +6,7 @@ from __future__ import annotations
 
 import torch
 
+from ..weights.loader import TensorSpec
 from .registry import register_block
 from .runtime import Runtime
 
@@ -191,8 +192,12 @@ class SandwichBlock:
     into the zeroed buffer, so every registered mixer and feed-forward fits); one kernel norms that output,
     adds it to the stream and applies the norm that comes next (this block's second, or the next block's
     first, which is handed on as a `NormedInput`), so the stream crosses memory once per sublayer.  The
-    fused kernel takes norms with a plain weight per coordinate (`weight`, `eps`); the next norm is fused
-    only if its weight has the same type as this one's."""
+    fused kernel takes norms with a plain weight per coordinate (`weight`, `eps`), and layer norms (`bias`
+    too); the next norm is fused only if it is of the same kind and its weight has the same type as this one's.
+
+    Optional parameters: `scales`, the names under `prefix` of one vector per sublayer (of `size` numbers) that
+    multiplies what the sublayer's output norm gives.  They are taken into that norm's weight and bias when the
+    weights come in (32-bit)."""
     norm_roles = ("mixer_norm", "mixer_out_norm", "feed_forward_norm", "feed_forward_out_norm")
     takes_carry = True
 
@@ -201,14 +206,30 @@ class SandwichBlock:
         self.mixer = mixer
         self.feed_forward = feed_forward
         self.norms = dict(norms)
+        self.scales = tuple(spec.get("scales") or ())
+        self.prefix = str(spec.get("prefix") or "")
+        self._scaled = {}        # output norm's role -> (weight, bias) with the sublayer's scale in them
+
+    @classmethod
+    def expected_tensors(cls, spec, prefix: str):
+        return {f"{prefix}.{n}": TensorSpec((int(spec.params["size"]),)) for n in (spec.get("scales") or ())}
+
+    def load(self, weights) -> None:
+        for role, name in zip(("mixer_out_norm", "feed_forward_out_norm"), self.scales):
+            norm = self.norms[role]
+            s = weights[f"{self.prefix}.{name}"].to(device=self.rt.device, dtype=torch.float32)
+            bias = getattr(norm, "bias", None)
+            self._scaled[role] = ((norm.weight.to(torch.float32) * s).contiguous(),
+                                  (bias * s).contiguous() if bias is not None else None)
 
     @property
     def first_norm(self):
         return self.norms["mixer_norm"]
 
-    def _sublayer(self, part, norm_in, norm_out, x, xn, batch, next_norm):
-        """x += norm_out(part(xn)); returns next_norm(x) if it could be taken along, else None."""
-        rt = self.rt
+    def _sublayer(self, part, role, x, xn, batch, next_norm):
+        """x += norms[role](part(xn)); returns next_norm(x) if it could be taken along, else None."""
+        rt, norm_out = self.rt, self.norms[role]
+        weight, bias = self._scaled.get(role) or (norm_out.weight, getattr(norm_out, "bias", None))
         y = rt.workspace.get("branch_out", x.shape, torch.float32)
         if getattr(part, "can_overwrite", False):
             part.forward(xn, y, batch, overwrite=True)
@@ -217,12 +238,14 @@ class SandwichBlock:
             part.forward(xn, y, batch)
         fuse = (next_norm is not None and getattr(next_norm, "weight", None) is not None
                 and getattr(next_norm, "size", None) == x.shape[1]
-                and next_norm.weight.dtype == norm_out.weight.dtype)
-        if not fuse:
-            rt.ops.norm_add_norm(y, norm_out.weight, norm_out.eps, x)
-            return None
-        out = rt.workspace.get("block_normed", x.shape, rt.act_dtype)
-        rt.ops.norm_add_norm(y, norm_out.weight, norm_out.eps, x, next_norm.weight, next_norm.eps, out)
+                and next_norm.weight.dtype == weight.dtype
+                and (getattr(next_norm, "bias", None) is None) == (bias is None))
+        out = rt.workspace.get("block_normed", x.shape, rt.act_dtype) if fuse else None
+        if bias is not None:
+            then = (next_norm.weight, next_norm.bias, next_norm.eps, out) if fuse else ()
+            rt.ops.layernorm_add_layernorm(y, weight, bias, norm_out.eps, x, *then)
+        else:
+            rt.ops.norm_add_norm(y, weight, norm_out.eps, x, *((next_norm.weight, next_norm.eps, out) if fuse else ()))
         return out
 
     def _input(self, norm, x, carry):
@@ -234,12 +257,11 @@ class SandwichBlock:
         n = self.norms
         xn = self._input(n["mixer_norm"], x, carry)
         second = n.get("feed_forward_norm")
-        got = self._sublayer(self.mixer, n["mixer_norm"], n["mixer_out_norm"], x, xn, batch,
-                             second if second is not None else next_norm)
+        got = self._sublayer(self.mixer, "mixer_out_norm", x, xn, batch, second if second is not None else next_norm)
         if second is None:
             return NormedInput(got, next_norm) if got is not None else None
         xn = got if got is not None else second(x, self.rt.workspace.get("block_normed", x.shape, self.rt.act_dtype))
-        got = self._sublayer(self.feed_forward, second, n["feed_forward_out_norm"], x, xn, batch, next_norm)
+        got = self._sublayer(self.feed_forward, "feed_forward_out_norm", x, xn, batch, next_norm)
         return NormedInput(got, next_norm) if got is not None else None
 
 

@@ -1,5 +1,6 @@
 """RMSNorm: y = x / sqrt(mean(x^2) + eps) * w, computed in 32-bit
-(reference: src/kernels/mod.rs:558-568, src/model/modules/rmsnorm.rs:6-25)."""
+(reference: src/kernels/mod.rs:558-568, src/model/modules/rmsnorm.rs:6-25), two variants of its weight, and
+the layer norm."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -99,4 +100,33 @@ class OnePlusRMSNorm:
 
     def __call__(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         self.rt.ops.rmsnorm(x, self.weight, self.eps, out, rows)
+        return out
+
+
+@register_norm("layernorm")
+class LayerNorm:
+    """y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w + b.  Parameters: `size`, `eps`.  Tensors: the
+    weight under the norm's own name, the bias under that name with `.b`.  `weight` and `bias` are 32-bit."""
+
+    foldable = False
+
+    def __init__(self, spec: PartSpec, prefix: str, rt: Runtime):
+        self.size = int(spec.params["size"])
+        self.eps = float(spec.params["eps"])
+        self.name = prefix
+        self.rt = rt
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    @classmethod
+    def expected_tensors(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorSpec]:
+        size = int(spec.params["size"])
+        return {prefix: TensorSpec((size,)), f"{prefix}.b": TensorSpec((size,), init=(0.1, 0.0))}
+
+    def load(self, weights: Dict[str, torch.Tensor]) -> None:
+        f32 = lambda t: t.to(device=self.rt.device, dtype=torch.float32).contiguous()
+        self.weight, self.bias = f32(weights[self.name]), f32(weights[f"{self.name}.b"])
+
+    def __call__(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        self.rt.ops.layernorm(x, self.weight, self.bias, self.eps, out, rows)
         return out

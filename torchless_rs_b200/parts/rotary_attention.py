@@ -21,6 +21,9 @@ divided by their root mean square after the rotation if asked,
     score = scale (q_i . k_j),   j visible iff 0 <= i - j < window,
     p(i, j) = exp(score(i, j)) / (sum over visible j' of exp(score(i, j')) + exp(sink_head))
     out = W_o (concatenated heads) + b_o
+Its values may be mixed with those of an earlier layer (`value_mix`): the layer called "first" leaves its
+projected values where the others find them, the ones called "later" cache (1 - l) v + l v_first, l their own
+learned number and v_first the same token's values of the "first" one.
 
 All: one stacked product for the projections of the input (32-bit), one kernel that rotates, norms
 and writes q and the token's k and v into the pages, attention from pages only (so a position's
@@ -52,6 +55,8 @@ class _RotaryAttention:
     plain_scores = True  # nothing but the keys enters the softmax (False: a sink does; the plain kernels are not built)
     proj_bias = None     # 32-bit, one number per column of the stacked projections (None: no bias)
     values_are_keys = False   # no value projection: a head's values are its keys as projected
+    value_mix = None          # "first": leave the values for later layers; "later": mix them with the first's
+    mix_weight = 0.0
 
     def __init__(self, spec: PartSpec, prefix: str, rt: Runtime, position=None):
         p = spec.params
@@ -103,10 +108,13 @@ class _RotaryAttention:
         self.matmul(xn, self.w_in, z, ops.MODE_STORE_F32)
         q = ws.get("rot_attn_q", (T, H * S * self.width), rt.act_dtype)
         pos = self.position
+        first_values = ws.get("value_mix_first", (T, G * self.vdim), torch.float32) if self.value_mix else None
         rt.ops.rotary_cache_write(z, pos.inv_freq if self.rot else None, self.rot, pos.style if self.rot else 0,
                                   self.unit_norm, self.eps, q, c.k_pages, c.v_pages, batch.token_pos,
                                   batch.token_seq, batch.seq_slot, c.page_table, H * S, G * S, G, self.dim,
-                                  self.vdim, S, bias=self.proj_bias, values_are_keys=self.values_are_keys)
+                                  self.vdim, S, bias=self.proj_bias, values_are_keys=self.values_are_keys,
+                                  amplitude=getattr(pos, "amplitude", 1.0), first_values=first_values,
+                                  mix=self.mix_weight if self.value_mix == "later" else None)
         return z, q
 
     def _attend(self, q, out, batch, softcap, sink=None):
@@ -216,8 +224,10 @@ class SinkRotaryAttention(_RotaryAttention):
     """Parameters: `hidden_size`, `heads`, `kv_heads`, `dim`, `vdim`, `rot_dims`, `scale`, `window` (None: all
     keys), `eps` (of the query and key norms), `unit_norm` (queries and keys divided by their root mean square
     after the rotation), `sink` (a learned logit per head in the denominator), `bias` (q, k, v and o have
-    biases, stored under the tensor's name with `.b`), `values_are_keys` (no v: `vdim` must equal `dim`).
-    Tensors under the prefix: q, k, [v], o, [q.b, k.b, v.b, o.b], [sink].
+    biases, stored under the tensor's name with `.b`), `values_are_keys` (no v: `vdim` must equal `dim`),
+    `value_mix` (None, "first" or "later": the values of several layers mixed, see the module's text).
+    Tensors under the prefix: q, k, [v], o, [q.b, k.b, v.b, o.b], [sink], [vmix] (one number; stored but not used
+    where `value_mix` is "first").
 
     `output_bias` is the output projection's bias (or None); `forward(..., defer_bias=True)` leaves it out, for
     a caller that adds it where it sums this mixer's output with others'."""
@@ -229,6 +239,9 @@ class SinkRotaryAttention(_RotaryAttention):
         self.plain_scores = not bool(p.get("sink", False))
         super().__init__(spec, prefix, rt, position)
         self.window = int(p["window"]) if p.get("window") else None
+        self.value_mix = p.get("value_mix")
+        if self.value_mix not in (None, "first", "later"):
+            raise ValueError(f"'value_mix' is 'first', 'later' or absent, not '{self.value_mix}'")
         self.has_sink = bool(p.get("sink", False))
         self.has_bias = bool(p.get("bias", False))
         if self.values_are_keys and self.vdim != self.dim:
@@ -254,6 +267,8 @@ class SinkRotaryAttention(_RotaryAttention):
                 out[f"{prefix}.v.b"] = TensorSpec((G * vdim,), init=(0.1, 0.0))
         if p.get("sink"):
             out[f"{prefix}.sink"] = TensorSpec((H,), init=(1.0, 0.0))
+        if p.get("value_mix"):
+            out[f"{prefix}.vmix"] = TensorSpec((), init=(0.1, 0.5), optional=p["value_mix"] == "first")
         return out
 
     def load(self, weights: Dict[str, torch.Tensor]) -> None:
@@ -267,6 +282,8 @@ class SinkRotaryAttention(_RotaryAttention):
             self.output_bias = f32(weights[f"{p}.o.b"])
         if self.has_sink:
             self.sink = f32(weights[f"{p}.sink"])
+        if self.value_mix == "later":
+            self.mix_weight = float(weights[f"{p}.vmix"].to(torch.float32))
 
     def forward(self, xn: torch.Tensor, residual: torch.Tensor, batch, emit=None, overwrite: bool = False,
                 defer_bias: bool = False) -> None:
