@@ -280,10 +280,10 @@ def reference_arm(args) -> int:
 
 
 def design_arm(args) -> int:
-    """`--design kikopel|tovapel|rupasun|fezolorn|dunesun`: prefill and decode throughput of that design at layer sizes
+    """`--design kikopel|tovapel|rupasun|fezolorn|dunesun|beralix`: prefill and decode throughput of that design at layer sizes
     of a real model (random weights), beside the closest existing model (Mistral; for fezolorn the third design, whose
     layers also run attention with a sink beside a linear recurrence; for dunesun the fourth, with windowed attention
-    and chosen and shared experts in every layer) at equal width, heads, layers, feed-forward and window, and every
+    and chosen and shared experts in every layer; for beralix the second, with latent attention and a recurrence) at equal width, heads, layers, feed-forward and window, and every
     kernel of the design alone against its roofline beside the like kernel of an existing path.  One JSON line; the default workload is not touched."""
     import torch
     import torchless_rs_b200 as tl
@@ -295,12 +295,13 @@ def design_arm(args) -> int:
     design = args.design
     sizes = {"kikopel": measure.KIKOPEL_SIZES, "tovapel": measure.TOVAPEL_SIZES,
              "rupasun": measure.RUPASUN_SIZES, "fezolorn": measure.FEZOLORN_SIZES,
-             "dunesun": measure.DUNESUN_SIZES}[design]
+             "dunesun": measure.DUNESUN_SIZES, "beralix": measure.BERALIX_SIZES}[design]
     configs = {"kikopel": (measure.kikopel_config, measure.mistral_like, measure.kikopel_kernels),
                "tovapel": (measure.tovapel_config, measure.tovapel_like, measure.tovapel_kernels),
                "rupasun": (measure.rupasun_config, measure.rupasun_like, measure.rupasun_kernels),
                "fezolorn": (measure.fezolorn_config, measure.fezolorn_like, measure.fezolorn_kernels),
-               "dunesun": (measure.dunesun_config, measure.dunesun_like, measure.dunesun_kernels)}[design]
+               "dunesun": (measure.dunesun_config, measure.dunesun_like, measure.dunesun_kernels),
+               "beralix": (measure.beralix_config, measure.beralix_like, measure.beralix_kernels)}[design]
     out = {"design": design, "sizes": dict(sizes[size]), "layers": L, "dtype": "bf16",
            "data": "synthetic: random weights, fixed token ids", "prefill_tokens": T, "decode_batch": B,
            "decode_context": ctx, "steps": args.steps, "warmup": args.warmup}
@@ -348,7 +349,7 @@ def design_arm(args) -> int:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["kikopel", "tovapel", "rupasun", "fezolorn", "dunesun"],
+    ap.add_argument("--design", default=None, choices=["kikopel", "tovapel", "rupasun", "fezolorn", "dunesun", "beralix"],
                     help="measure another design beside Mistral at equal sizes instead of the default workload")
     ap.add_argument("--design-size", default="1b", choices=["1b", "7b"])
     ap.add_argument("--gpus", type=int, default=1)

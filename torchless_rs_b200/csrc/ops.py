@@ -143,7 +143,7 @@ class CoreOps:
                      "tl_clamped_glu", "tl_delta_prep", "tl_conv_state_update", "tl_delta_scan", "tl_silu_rows",
                      "tl_weighted_sum", "tl_close_block", "tl_moe_route_chosen", "tl_qk_whole_norm_cache_write",
                      "tl_ssd_prep", "tl_ssd_walk", "tl_ssd_gate_norm", "tl_layernorm",
-                     "tl_layernorm_add_layernorm", "tl_selective_scan"):
+                     "tl_layernorm_add_layernorm", "tl_selective_scan", "tl_conv_silu"):
             fn = getattr(self.lib, f"{base}_{self.suffix}")
             fn.restype = c_int
             setattr(self, "_" + base, fn)
@@ -1223,8 +1223,8 @@ class CoreOps:
     def conv_silu(self, z: torch.Tensor, col: int, taps_w: torch.Tensor, bias: torch.Tensor, kept: torch.Tensor,
                   out: torch.Tensor, seq_start: torch.Tensor, seq_slot: torch.Tensor) -> None:
         """out [T, channels] = silu(conv(z[:, col:]) + bias), the convolution and its kept inputs as in `ssd_prep`
-        (whose kernel this is, without step sizes)."""
-        _need(z, torch.float32, "projections", contiguous=False)
+        (whose kernel this is, without step sizes); z in the activation type."""
+        _need(z, self.act_dtype, "projections", contiguous=False)
         _need(out, self.act_dtype, "convolved channels")
         for t, n in ((taps_w, "convolution taps"), (bias, "convolution bias"), (kept, "kept convolution inputs")):
             _need(t, torch.float32, n)
@@ -1233,10 +1233,9 @@ class CoreOps:
         if z.stride(1) != 1 or z.shape[0] != T or z.shape[1] < col + channels or taps_w.shape != (channels, taps) or \
                 bias.numel() != channels or kept.shape[2] != channels or kept.shape[1] != max(taps - 1, 1):
             raise KernelError("conv_silu: sizes do not match")
-        _check(self._tl_ssd_prep(_ptr(z), c_int(z.stride(0)), c_int(col), c_int(0), _ptr(taps_w), _ptr(bias),
-                                 c_int(taps), _ptr(kept), _ptr(out), _ptr(None), _ptr(None), _ptr(None),
-                                 _ptr(seq_start), _ptr(seq_slot), c_int(T), c_int(seq_slot.numel()), c_int(channels),
-                                 c_int(0), _stream()), "conv_silu")
+        _check(self._tl_conv_silu(_ptr(z), c_int(z.stride(0)), c_int(col), _ptr(taps_w), _ptr(bias), c_int(taps),
+                                  _ptr(kept), _ptr(out), _ptr(seq_start), _ptr(seq_slot), c_int(T),
+                                  c_int(seq_slot.numel()), c_int(channels), _stream()), "conv_silu")
 
     def selective_scan(self, x: torch.Tensor, zdt: torch.Tensor, dt_bias: torch.Tensor, bc: torch.Tensor, col_b: int,
                        neg_a: torch.Tensor, D: torch.Tensor, z: torch.Tensor, state: torch.Tensor, y: torch.Tensor,
@@ -1250,7 +1249,7 @@ class CoreOps:
         for t, n in ((zdt, "step sizes"), (dt_bias, "step size bias"), (neg_a, "decay rates"), (D, "skip weights"),
                      (state, "recurrent state")):
             _need(t, torch.float32, n)
-        _need(z, torch.float32, "gate", contiguous=False)
+        _need(z, self.act_dtype, "gate", contiguous=False)
         T, channels = x.shape
         N = neg_a.shape[1]
         if zdt.shape != (T, channels) or dt_bias.numel() != channels or bc.shape[0] != T or bc.shape[1] < col_b + 2 * N or \

@@ -3,7 +3,7 @@
 //   dt = softplus(zdt_c + b_c),   S_c,n <- exp(dt A_c,n) S_c,n + dt x_c B_n,
 //   y_c = (sum_n S_c,n C_n + D_c x_c) * silu(z_c)                                    (A < 0, given)
 // over each sequence's tokens of the step, from and into the state in the sequence's slot (32-bit).  Step sizes,
-// decays, state, sums and the gate are 32-bit; x, B and C come in the activation type, y leaves in it.
+// decays, state, sums and the gate are 32-bit; x, z, B and C come in the activation type, y leaves in it.
 //
 // A block owns (sequence, a run of channels); a channel's states lie in the registers of LPC neighbouring lanes,
 // NS each (padded with states that stay zero), so a token costs a thread NS exponentials, NS multiply-adds for the state and NS for the output, and
@@ -70,13 +70,13 @@ __device__ __forceinline__ void sc_read(const float* p, float (&v)[NS]) {
   }
 }
 
-// x: [T, ldx]; zdt: [T, channels] 32-bit; bc: [T, ldbc] with B at column col_b and C at col_b + N; z: [T, ldz]
-// 32-bit; A: [channels, N]; state: [slots, channels, N]; y: [T, channels].
+// x: [T, ldx]; zdt: [T, channels] 32-bit; bc: [T, ldbc] with B at column col_b and C at col_b + N; z: [T, ldz];
+// A: [channels, N]; state: [slots, channels, N]; y: [T, channels].
 template <int LPC, int NS, int TT>
 __global__ void __launch_bounds__(SC_THREADS)
 selective_scan_kernel(const act_t* __restrict__ x, int ldx, const float* __restrict__ zdt,
                       const float* __restrict__ dt_bias, const act_t* __restrict__ bc, int ldbc, int col_b,
-                      const float* __restrict__ A, const float* __restrict__ D, const float* __restrict__ z, int ldz,
+                      const float* __restrict__ A, const float* __restrict__ D, const act_t* __restrict__ z, int ldz,
                       float* __restrict__ state, act_t* __restrict__ y, const int* __restrict__ seq_start,
                       const int* __restrict__ seq_slot, int channels, int N) {
   constexpr int CH = SC_THREADS / LPC;            // channels of a block
@@ -116,7 +116,7 @@ selective_scan_kernel(const act_t* __restrict__ x, int ldx, const float* __restr
       const bool ok = live && et + k * ET < TT && t < t1;
       rdt[k] = ok ? zdt[(size_t)t * channels + c0 + ec] : 0.0f;
       nx[k] = ok ? to_f32(x[(size_t)t * ldx + c0 + ec]) : 0.0f;
-      nz[k] = ok ? z[(size_t)t * ldz + c0 + ec] : 0.0f;
+      nz[k] = ok ? to_f32(z[(size_t)t * ldz + c0 + ec]) : 0.0f;
     }
     if (AHEAD) {
 #pragma unroll
@@ -199,7 +199,7 @@ selective_scan_kernel(const act_t* __restrict__ x, int ldx, const float* __restr
 
 extern "C" int TL_NAME(tl_selective_scan)(const void* x, int ldx, const float* zdt, const float* dt_bias,
                                           const void* bc, int ldbc, int col_b, const float* A, const float* D,
-                                          const float* z, int ldz, float* state, void* y, const int* seq_start,
+                                          const void* z, int ldz, float* state, void* y, const int* seq_start,
                                           const int* seq_slot, int B, int channels, int N, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (channels < 1 || N < 1 || col_b < 0) return TL_ERR_BAD_ARG;
@@ -207,7 +207,7 @@ extern "C" int TL_NAME(tl_selective_scan)(const void* x, int ldx, const float* z
 #define SCAN(LPC_, NS_, TT_)                                                                                         \
   return tl_launch(selective_scan_kernel<LPC_, NS_, TT_>, dim3((channels + SC_THREADS / LPC_ - 1) / (SC_THREADS / LPC_), B), \
                    dim3(SC_THREADS), 0, stream, (const act_t*)x, ldx, zdt, dt_bias, (const act_t*)bc, ldbc, col_b, A,  \
-                   D, z, ldz, state, (act_t*)y, seq_start, seq_slot, channels, N)
+                   D, (const act_t*)z, ldz, state, (act_t*)y, seq_start, seq_slot, channels, N)
   if (N <= 4) SCAN(1, 4, 16);
   if (N <= 8) SCAN(2, 4, 16);
   if (N <= 16) SCAN(4, 4, 16);

@@ -8,6 +8,7 @@
 //   ssd_prep         the step's projections -> convolved, activated x, B, C (activation type), dt and the
 //                    decay's logarithm per token and head (32-bit); the last taps - 1 inputs go back to
 //                    the sequence's slot
+//   conv_silu        the convolution alone, on inputs of the activation type
 //   ssd_walk         the recurrence token by token from the state in the slot: decode steps, short steps
 //                    and the whole of the 32-bit path
 //   ssd_chunk_state, ssd_chunk_carry, ssd_chunk_out
@@ -57,9 +58,9 @@ __device__ __forceinline__ bool ssd_find_piece(int id, int size, const int* seq_
 // A thread per channel walks a strip of 16 tokens; the thread of a sequence's first strip, the only one that
 // looks at the kept inputs, also replaces them.  The blocks past the channels' take the step sizes.
 // TAPS: the number of taps, or 0 for any (their inputs are then read where they are needed).
-template <int TAPS>
+template <int TAPS, typename Z>
 __global__ void __launch_bounds__(128)
-ssd_prep_kernel(const float* __restrict__ z, int ld, int col_x, int col_dt, const float* __restrict__ taps_w,
+ssd_prep_kernel(const Z* __restrict__ z, int ld, int col_x, int col_dt, const float* __restrict__ taps_w,
                 const float* __restrict__ bias, int taps_rt, float* __restrict__ kept, act_t* __restrict__ xbc,
                 float2* __restrict__ dtla, const float* __restrict__ neg_a, const float* __restrict__ dt_bias,
                 const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int B, int channels, int H,
@@ -73,20 +74,20 @@ ssd_prep_kernel(const float* __restrict__ z, int ld, int col_x, int col_dt, cons
     for (int i = threadIdx.x + ((int)blockIdx.y - ch_blocks) * blockDim.x; i < n * H;
          i += (gridDim.y - ch_blocks) * blockDim.x) {
       const int t = t0 + i / H, h = i % H;
-      const float dt = ssd_softplus(z[(size_t)t * ld + col_dt + h] + dt_bias[h]);
+      const float dt = ssd_softplus(to_f32(z[(size_t)t * ld + col_dt + h]) + dt_bias[h]);
       dtla[(size_t)t * H + h] = make_float2(dt, neg_a[h] * dt);
     }
     return;
   }
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= channels) return;
-  const float* zc = z + col_x + c;
+  const Z* zc = z + col_x + c;
   float* mine = kept + (size_t)seq_slot[b] * (taps - 1) * channels + c;
   const float bi = bias[c];
   const int first = seq_start[b], count = seq_start[b + 1] - first, j0 = strip * SSD_STRIP;
   // the input at place j of the step (j < 0: kept from before)
   auto input = [&](int j) -> float {
-    return j >= 0 ? zc[(size_t)(first + j) * ld] : mine[(size_t)(taps - 1 + j) * channels];
+    return j >= 0 ? to_f32(zc[(size_t)(first + j) * ld]) : mine[(size_t)(taps - 1 + j) * channels];
   };
   if (TAPS) {
     float v[SSD_STRIP + (TAPS ? TAPS : 1) - 1], w[TAPS ? TAPS : 1];
@@ -121,19 +122,20 @@ ssd_prep_kernel(const float* __restrict__ z, int ld, int col_x, int col_dt, cons
   }
 }
 
-extern "C" int TL_NAME(tl_ssd_prep)(const float* z, int ld, int col_x, int col_dt, const float* taps_w,
-                                    const float* bias, int taps, float* kept, void* xbc, float* dtla,
-                                    const float* neg_a, const float* dt_bias, const int* seq_start,
-                                    const int* seq_slot, int T, int B, int channels, int H, cudaStream_t stream) {
+template <typename Z>
+static int ssd_prep_launch(const Z* z, int ld, int col_x, int col_dt, const float* taps_w, const float* bias, int taps,
+                           float* kept, void* xbc, float* dtla, const float* neg_a, const float* dt_bias,
+                           const int* seq_start, const int* seq_slot, int T, int B, int channels, int H,
+                           cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
-  if (channels < 1 || H < 0 || taps < 1) return TL_ERR_BAD_ARG;     // H = 0: the convolution alone
+  if (channels < 1 || H < 0 || taps < 1) return TL_ERR_BAD_ARG;
   if (taps > SSD_MAX_TAPS) return TL_ERR_UNSUPPORTED;
   const int ch_blocks = (channels + 127) / 128;
   const int dt_blocks = (H * (T < SSD_STRIP ? T : SSD_STRIP) + 511) / 512;
   dim3 grid(T / SSD_STRIP + B, ch_blocks + dt_blocks);
   if (grid.y > 65535) return TL_ERR_UNSUPPORTED;
 #define PREP(TAPS_)                                                                                            \
-  return tl_launch(ssd_prep_kernel<TAPS_>, grid, dim3(128), 0, stream, z, ld, col_x, col_dt, taps_w, bias, taps, \
+  return tl_launch(ssd_prep_kernel<TAPS_, Z>, grid, dim3(128), 0, stream, z, ld, col_x, col_dt, taps_w, bias, taps, \
                    kept, (act_t*)xbc, (float2*)dtla, neg_a, dt_bias, seq_start, seq_slot, B, channels, H, ch_blocks)
   switch (taps) {
     case 1: PREP(1);
@@ -143,6 +145,23 @@ extern "C" int TL_NAME(tl_ssd_prep)(const float* z, int ld, int col_x, int col_d
     default: PREP(0);
   }
 #undef PREP
+}
+
+extern "C" int TL_NAME(tl_ssd_prep)(const float* z, int ld, int col_x, int col_dt, const float* taps_w,
+                                    const float* bias, int taps, float* kept, void* xbc, float* dtla,
+                                    const float* neg_a, const float* dt_bias, const int* seq_start,
+                                    const int* seq_slot, int T, int B, int channels, int H, cudaStream_t stream) {
+  if (H < 1) return TL_ERR_BAD_ARG;
+  return ssd_prep_launch<float>(z, ld, col_x, col_dt, taps_w, bias, taps, kept, xbc, dtla, neg_a, dt_bias, seq_start,
+                                seq_slot, T, B, channels, H, stream);
+}
+
+// The convolution alone: out [T, channels] = silu(conv(z[:, col_x:]) + bias), z in the activation type.
+extern "C" int TL_NAME(tl_conv_silu)(const void* z, int ld, int col_x, const float* taps_w, const float* bias, int taps,
+                                     float* kept, void* out, const int* seq_start, const int* seq_slot, int T, int B,
+                                     int channels, cudaStream_t stream) {
+  return ssd_prep_launch<act_t>((const act_t*)z, ld, col_x, 0, taps_w, bias, taps, kept, out, nullptr, nullptr, nullptr,
+                                seq_start, seq_slot, T, B, channels, 0, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------

@@ -1124,6 +1124,215 @@ def dunesun_kernels(size: str, T: int, B: int, ctx: int, iters: int, file=None) 
     return rows
 
 
+# Layer sizes at which the Beralix kernels are measured: the width, heads and feed-forward of a 1B- and a
+# 7B-class decoder; window attention with a quarter as many key/value heads and a window of 1024, latents of the
+# sizes of the second design with queries straight from the input, a selective scan over twice the width with 16
+# state entries per channel and step sizes through a sixteenth of the width (as published models have it).
+BERALIX_SIZES = {
+    "1b": dict(width=2048, heads=16, kv_heads=4, dim=128, window=1024, ff=5632, m_heads=16, m_dim=128, m_rot=64,
+               m_vdim=128, kv_rank=512, inner=4096, state=16, dt_rank=128, conv=4, vocab=32000),
+    "7b": dict(width=4096, heads=32, kv_heads=8, dim=128, window=1024, ff=14336, m_heads=32, m_dim=128, m_rot=64,
+               m_vdim=128, kv_rank=512, inner=8192, state=16, dt_rank=256, conv=4, vocab=32000),
+}
+
+
+def beralix_config(size: str, layers: int) -> dict:
+    """config.json of a Beralix model of `layers` layers at these sizes: window attention, latent attention,
+    selective scan, latent attention in turn."""
+    z = BERALIX_SIZES[size]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    scaling = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "v_mix": True,
+        "scale": 1.0 / math.sqrt(z["dim"]), "mask": {"size": z["window"]},
+        "rot": {"base": 500000.0, "dims": z["dim"], "scaling": scaling}}}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": z["m_heads"], "dim": z["m_dim"], "rot_dim": z["m_rot"], "vdim": z["m_vdim"], "kv_rank": z["kv_rank"],
+        "rot": {"base": 500000.0, "dims": z["m_rot"], "scaling": scaling},
+        "scale": 1.0 / math.sqrt(z["m_dim"] + z["m_rot"])}}
+    ssm = {"type": "mamba1", "mlp": mlp, "mixer": {k: z[k] for k in ("inner", "state", "dt_rank", "conv")}}
+    return {"architecture": "Beralix", "width": z["width"], "vocab": z["vocab"], "norm": {"eps": 1e-5},
+            "logit_softcap": 30.0, "max_position_embeddings": 32768,
+            "layers": [(att, lat, ssm, lat)[i % 4] for i in range(layers)]}
+
+
+def beralix_like(size: str, layers: int) -> dict:
+    """The closest existing model at equal size: the second design (latent attention, a recurrence, a norm on every
+    sublayer's output) with the same width, heads, feed-forward and latent, its latent attention with the window
+    where the design has window attention, its recurrence where the design has the selective scan."""
+    z, k = BERALIX_SIZES[size], KIKOPEL_SIZES[size]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+
+    def att(window):
+        return {"type": "latent_attention", "mlp": mlp, "mixer": {
+            "heads": z["m_heads"], "dim": z["m_dim"], "rot_dim": z["m_rot"], "vdim": z["m_vdim"], "q_rank": k["q_rank"],
+            "kv_rank": z["kv_rank"], "mask": {"size": window}, "rot": {"base": 500000.0, "dims": z["m_rot"]},
+            "scale": 1.0 / math.sqrt(z["m_dim"] + z["m_rot"])}}
+    rec = {"type": "hgrn2", "mlp": mlp, "mixer": {"heads": k["r_heads"], "dim": k["r_dim"], "vdim": k["r_vdim"]}}
+    return {"architecture": "Kikopel", "width": z["width"], "vocab": z["vocab"], "norm": {"eps": 1e-5},
+            "residual_mult": 0.6, "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 131}},
+            "layers": [(att(z["window"]), att(32768), rec, att(32768))[i % 4] for i in range(layers)],
+            "max_position_embeddings": 32768}
+
+
+def beralix_kernels(size: str, T: int, B: int, ctx: int, iters: int, file=None) -> list:
+    """Every kernel that the Beralix design added or changed, alone at the sizes `size`, for a prompt of T tokens
+    and for a decode step of B sequences at a context of `ctx`, beside the like kernel of an existing model at
+    equal sizes.  Rows and roofline as `kikopel_kernels` defines them."""
+    import json
+    import os
+    from .csrc import ops
+    from .csrc.attention_bf16 import AttentionBf16
+    from .parts.runtime import Workspace
+    z = BERALIX_SIZES[size]
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    pk = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
+    if os.path.isfile(pk):
+        peaks.update(json.load(open(pk)))
+    o = ops.core_ops(torch.bfloat16)
+    dev, bf = "cuda", torch.bfloat16
+    H, G, dim, W = z["heads"], z["kv_heads"], z["dim"], z["width"]
+    rows = []
+
+    def report(name, case, us, byts, flops):
+        t_mem, t_fl = byts / (peaks["hbm_gbs"] * 1e3), flops / (peaks["bf16_tflops"] * 1e6)     # microseconds
+        frac = max(t_mem, t_fl) / us
+        rows.append({"kernel": name, "case": case, "us": round(us, 2), "roofline_frac": round(frac, 4),
+                     "bound": "memory" if t_mem >= t_fl else "tensor"})
+        print(f"{name:42s} {case:18s} {us:10.2f} us   {frac:7.4f} of the roofline ({rows[-1]['bound']})", file=file)
+
+    ws = Workspace(torch.device("cuda"))
+    for case, n_tok, seqs, past in ((f"prompt {T}", T, 1, 0), (f"decode {B} x {ctx}", B, B, ctx - 1)):
+        per = n_tok // seqs
+        few = max(2, iters // 8) if n_tok > 64 else iters
+        pos = torch.cat([torch.arange(past, past + per, dtype=torch.int32) for _ in range(seqs)]).to(dev)
+        seq = torch.arange(seqs, dtype=torch.int32).repeat_interleave(per).to(dev)
+        start = (torch.arange(seqs + 1, dtype=torch.int32) * per).to(dev)
+        # --- window attention: the rotation with its amplitude and the mixed values; the attention is Mistral's
+        kp, vp, table, slot = _paged(seqs, past + per, G, dim)
+        lens = torch.full((seqs,), past + per, dtype=torch.int32, device=dev)
+        cols = (H + 2 * G) * dim
+        zq = torch.randn((n_tok, cols), device=dev)
+        q = torch.empty((n_tok, H * dim), device=dev, dtype=bf)
+        inv = torch.tensor([500000.0 ** (-2.0 * i / dim) for i in range(dim // 2)], device=dev)
+        first = torch.zeros((n_tok, G * dim), device=dev)
+        args = (zq, inv, dim, 0, False, 1e-5, q, kp, vp, pos, seq, slot, table, H, G, G, dim, dim)
+        us = _time(lambda: o.rotary_cache_write(*args, amplitude=1.2, first_values=first, mix=0.3), iters)
+        report("rotary_cache_write (mixed values)", case, us, n_tok * (cols * 6.0 + G * dim * 4.0), 0.0)
+        us = _time(lambda: o.rotary_cache_write(*args), iters)
+        report("  like: rotary_cache_write", case, us, n_tok * cols * 6.0, 0.0)
+        att = AttentionBf16.get(dim)
+        om = torch.empty_like(q)
+        seen = sum(min(p + 1, z["window"]) for p in range(past, past + per)) * seqs
+
+        class _B:      # what the kernel choice reads of a step
+            n_seqs, is_decode, len_bucket, max_new, seq_start, seq_len, seq_slot, new_lens = \
+                seqs, per == 1, past + per, per, start, lens, slot, [past + per] * seqs
+
+        class _C:      # the cache view of the attention kernels
+            k_pages, v_pages, page_table = kp, vp, table
+        us = _time(lambda: att.run(q, _C, om, _B, H, G, z["window"], 0.088, ws), iters)
+        report("attention (window, as Mistral's)", case, us,
+               2.0 * seqs * min(past + per, z["window"]) * G * 2 * dim + n_tok * H * dim * 4.0, 4.0 * H * dim * seen)
+        # --- latent attention
+        mh, md, rot, mv, rank = z["m_heads"], z["m_dim"], z["m_rot"], z["m_vdim"], z["kv_rank"]
+        q_rank = KIKOPEL_SIZES[size]["q_rank"]
+        width = rank + rot
+        n_pages = (past + per + 63) // 64
+        pages = torch.randn((seqs * n_pages, 64, width), device=dev, dtype=bf)
+        ltab = torch.arange(seqs * n_pages, dtype=torch.int32, device=dev).view(seqs, n_pages)
+        inv2 = torch.tensor([500000.0 ** (-2.0 * i / rot) for i in range(rot // 2)], device=dev)
+        qcols = mh * (md + rot)
+        s = torch.randn((n_tok, qcols + width + mh), device=dev)
+        wc, wq = torch.ones(rank, device=dev), torch.ones(q_rank, device=dev)
+        us = _time(lambda: o.latent_prep(None, s[:, qcols:qcols + width], None, wc, 1e-5, None, pages, pos, seq, slot, ltab,
+                                         inv2, rank, rot, rot, amplitude=1.2), iters)
+        report("latent_prep (no query latent)", case, us, n_tok * width * 6.0, 0.0)
+        s2 = torch.randn((n_tok, q_rank + width), device=dev)
+        cq = torch.empty((n_tok, q_rank), device=dev, dtype=bf)
+        us = _time(lambda: o.latent_prep(s2[:, :q_rank], s2[:, q_rank:], wq, wc, 1e-5, cq, pages, pos, seq, slot, ltab, inv2,
+                                         rank, rot, rot), iters)
+        report("  like: latent_prep", case, us, n_tok * (q_rank + width) * 6.0, 0.0)
+        wuk = torch.randn((mh, rank, md), device=dev, dtype=bf) * 0.02
+        wuv = torch.randn((mh, mv, rank), device=dev, dtype=bf) * 0.02
+        qa = torch.empty((n_tok, mh * rank), device=dev)
+        us = _time(lambda: o.headwise_gemm(s, md + rot, wuk, qa, rank), iters)
+        report("headwise_gemm (queries to latents)", case, us, mh * md * rank * 2.0 + n_tok * mh * (md + rank) * 4.0,
+               2.0 * n_tok * mh * md * rank)
+        mix = torch.randn((n_tok, mh, rank), device=dev)
+        og = torch.empty((n_tok, mh * mv), device=dev, dtype=bf)
+        us = _time(lambda: o.headwise_gemm(mix.view(n_tok, mh * rank), rank, wuv, og, mv, gate=s[:, qcols + width:]), iters)
+        report("headwise_gemm (values, gate per head)", case, us,
+               mh * mv * rank * 2.0 + n_tok * mh * (rank * 4.0 + mv * 2.0 + 4.0), 2.0 * n_tok * mh * mv * rank)
+        gate = torch.randn((n_tok, mh * mv), device=dev)
+        us = _time(lambda: o.headwise_gemm(mix.view(n_tok, mh * rank), rank, wuv, og, mv, gate=gate), iters)
+        report("  like: headwise_gemm (gate per entry)", case, us,
+               mh * mv * rank * 2.0 + n_tok * mh * (rank * 4.0 + mv * 6.0), 2.0 * n_tok * mh * mv * rank)
+        seen = sum(p + 1 for p in range(past, past + per)) * seqs
+        us = _time(lambda: o.latent_attn(qa, rank, s, md + rot, md, pages, mix, pos, seq, slot, ltab, inv2, mh, rank, rot, rot,
+                                         None, 0.04, max_keys=past + per, workspace=ws, amplitude=1.2), few)
+        byts = 2.0 * seqs * (past + per) * width + n_tok * mh * (width + rank) * 4.0
+        report("latent_attn", case, us, byts, 2.0 * mh * seen * (width + rank))
+        ql = torch.randn((n_tok, mh * width), device=dev)
+        us = _time(lambda: o.latent_attn(ql, width, ql, width, rank, pages, mix, pos, seq, slot, ltab, inv2, mh, rank, rot,
+                                         rot, None, 0.04, max_keys=past + per, workspace=ws), few)
+        report("  like: latent_attn (folded queries)", case, us, byts, 2.0 * mh * seen * (width + rank))
+        del ql, mix, s2, gate
+        # --- the selective scan, beside the second design's recurrence and the sixth's, each at an equal state
+        C, N, R, taps = z["inner"], z["state"], z["dt_rank"], z["conv"]
+        xz = torch.randn((n_tok, 2 * C), device=dev, dtype=bf)
+        x = torch.randn((n_tok, C), device=dev, dtype=bf)
+        kept = torch.zeros((seqs, taps - 1, C), device=dev)
+        tw, cb = torch.randn((C, taps), device=dev), torch.zeros(C, device=dev)
+        us = _time(lambda: o.conv_silu(xz, 0, tw, cb, kept, x, start, slot), iters)
+        report("conv_silu", case, us, n_tok * C * 4.0 + seqs * (taps - 1) * C * 8.0, 0.0)
+        dbc = torch.randn((n_tok, R + 2 * N), device=dev, dtype=bf)
+        zdt = torch.randn((n_tok, C), device=dev)
+        dtb, na, D = torch.zeros(C, device=dev) - 3.0, -torch.rand((C, N), device=dev), torch.ones(C, device=dev)
+        state = torch.zeros((seqs, C, N), device=dev)
+        y = torch.empty((n_tok, C), device=dev, dtype=bf)
+        us = _time(lambda: o.selective_scan(x, zdt, dtb, dbc, R, na, D, xz[:, C:], state, y, start, slot), few)
+        report("selective_scan", case, us, n_tok * (C * 10.0 + N * 4.0) + seqs * C * N * 8.0 + C * N * 4.0,
+               4.0 * n_tok * C * N)
+        P = 64
+        sh = C * N // (N * P)
+        ch = C + 2 * N
+        zz = torch.randn((n_tok, C + ch + sh), device=dev)
+        xbc = torch.empty((n_tok, ch), device=dev, dtype=bf)
+        dtla = torch.rand((n_tok, sh, 2), device=dev) * -0.1
+        kept2 = torch.zeros((seqs, taps - 1, ch), device=dev)
+        tw2, cb2 = torch.randn((ch, taps), device=dev), torch.zeros(ch, device=dev)
+        na2, dtb2, D2 = -torch.ones(sh, device=dev), torch.zeros(sh, device=dev), torch.ones(sh, device=dev)
+        state2 = torch.zeros((seqs, sh, N, P), device=dev)
+        so = torch.empty((n_tok, C), device=dev)
+        us = _time(lambda: o.ssd_prep(zz, C, C + ch, tw2, cb2, kept2, xbc, dtla, na2, dtb2, start, slot), iters)
+        report("  like: ssd_prep (convolution, steps)", case, us, n_tok * (ch * 6.0 + sh * 12.0) + seqs * (taps - 1) * ch * 8.0, 0.0)
+        us = _time(lambda: o.ssd_scan(xbc, dtla, D2, state2, so, start, slot, sh, 1, workspace=ws), few)
+        report("  like: ssd_scan (a decay per head)", case, us, n_tok * (ch * 2.0 + sh * 8.0 + C * 4.0) + seqs * C * N * 8.0,
+               4.0 * n_tok * C * N)
+        rv = 128
+        rh = max(1, C * N // (rv * rv))
+        z3 = torch.randn((n_tok, 3 * rh * rv), device=dev)
+        state3, so3 = torch.zeros((seqs, rh, rv, rv), device=dev), torch.empty((n_tok, rh * rv), device=dev)
+        bias, low = torch.zeros(rh * rv, device=dev), torch.full((rh * rv,), 0.5, device=dev)
+        us = _time(lambda: o.gated_scan(z3, bias, low, state3, so3, start, slot, rh, rv, rv, workspace=ws), few)
+        report("  like: gated_scan (equal state)", case, us, n_tok * 4 * rh * rv * 4.0 + seqs * rh * rv * rv * 8.0,
+               4.0 * n_tok * rh * rv * rv)
+        # --- the block's norms
+        xs, ys = torch.randn((n_tok, W), device=dev), torch.randn((n_tok, W), device=dev)
+        w1, b1, w2, b2 = (torch.randn(W, device=dev) for _ in range(4))
+        xn = torch.empty((n_tok, W), device=dev, dtype=bf)
+        us = _time(lambda: o.layernorm_add_layernorm(ys, w1, b1, 1e-5, xs, w2, b2, 1e-5, xn), iters)
+        report("layernorm_add_layernorm", case, us, n_tok * W * 14.0, 0.0)
+        us = _time(lambda: o.norm_add_norm(ys, w1, 1e-5, xs, w2, 1e-5, xn), iters)
+        report("  like: norm_add_norm", case, us, n_tok * W * 14.0, 0.0)
+        us = _time(lambda: o.layernorm(xs, w1, b1, 1e-5, xn), iters)
+        report("layernorm", case, us, n_tok * W * 6.0, 0.0)
+        us = _time(lambda: o.rmsnorm(xs, w1, 1e-5, xn), iters)
+        report("  like: rmsnorm", case, us, n_tok * W * 6.0, 0.0)
+    return rows
+
+
 def step(B: int, context: int, prefill: int, layers: int, iters: int) -> None:
     from . import from_random
     from .config import config_from_dict
@@ -1287,14 +1496,14 @@ def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("what", choices=["gemm", "attn-decode", "attn-prefill", "elementwise", "step", "timeline", "decode",
                                      "kikopel-kernels", "tovapel-kernels", "rupasun-kernels", "fezolorn-kernels",
-                                     "dunesun-kernels"])
+                                     "dunesun-kernels", "beralix-kernels"])
     ap.add_argument("sizes", type=int, nargs="+")
     ap.add_argument("--iters", type=int, default=50)
     ap.add_argument("--layers", type=int, default=4, help="layers of the model that `step` builds")
     ap.add_argument("--model", default="mistral7b", choices=sorted(MODEL_SIZES),
                     help="step, timeline: whose layer sizes the model has")
     ap.add_argument("--kikopel-size", default="1b", choices=sorted(KIKOPEL_SIZES),
-                    help="kikopel-kernels / tovapel-kernels / rupasun-kernels / fezolorn-kernels / dunesun-kernels "
+                    help="kikopel-kernels / tovapel-kernels / rupasun-kernels / fezolorn-kernels / dunesun-kernels / beralix-kernels "
                          "TOKENS BATCH CONTEXT: whose layer sizes the kernels get")
     ap.add_argument("--window", type=int, default=0, help="decode: the sliding window (0: none)")
     ap.add_argument("--equal-shares", action="store_true",
@@ -1312,6 +1521,9 @@ def main() -> None:
         return
     if a.what == "rupasun-kernels":
         rupasun_kernels(a.kikopel_size, a.sizes[0], a.sizes[1], a.sizes[2], a.iters)
+        return
+    if a.what == "beralix-kernels":
+        beralix_kernels(a.kikopel_size, a.sizes[0], a.sizes[1], a.sizes[2], a.iters)
         return
     if a.what == "dunesun-kernels":
         dunesun_kernels(a.kikopel_size, a.sizes[0], a.sizes[1], a.sizes[2], a.iters)

@@ -11,7 +11,7 @@ With h the mixer's input, per token (`inner` channels):
     out = W_o (y silu(z))
 S starts at zero, is 32-bit and is carried from token to token in the cache's per-sequence state together
 with the convolution's last `conv` - 1 inputs (two `StateRequest`s), so a prompt may come in any number of
-pieces.  Step sizes, decays and state are 32-bit; x, d, B and C are of the activation type.
+pieces.  Step sizes, decays, state and gate are 32-bit; x, z, d, B and C are of the activation type.
 
 The columns of d are padded to a multiple of 8 with zero rows of W_x and zero columns of W_dt, so that the
 second product reads its rows on 16-byte boundaries."""
@@ -95,8 +95,8 @@ class SelectiveScan:
     def forward(self, xn: torch.Tensor, residual: torch.Tensor, batch, emit=None, overwrite: bool = False) -> None:
         rt, ws = self.rt, self.rt.workspace
         T, inner = residual.shape[0], self.inner
-        xz = ws.get("scan1_in", (T, 2 * inner), torch.float32)
-        self.matmul(xn, self.w_in, xz, ops.MODE_STORE_F32)
+        xz = ws.get("scan1_in", (T, 2 * inner), rt.act_dtype)
+        self.matmul(xn, self.w_in, xz, ops.MODE_STORE_ACT)
         x = ws.get("scan1_x", (T, inner), rt.act_dtype)
         rt.ops.conv_silu(xz, 0, self.taps_w, self.conv_b, self.kept, x, batch.seq_start, batch.seq_slot)
         dbc = ws.get("scan1_dbc", (T, self.w_x.shape[0]), rt.act_dtype)
