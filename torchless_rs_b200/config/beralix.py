@@ -204,7 +204,7 @@ def _with_mix_roles(layers, where: str):
         if getattr(m, "v_mix", False):
             if first is None:
                 first = m
-            elif (m.kv_heads * m.vdim) != (first.kv_heads * first.vdim):
+            elif (m.kv_heads, m.vdim) != (first.kv_heads, first.vdim):
                 raise ConfigError(f"{where}: layers[{i}].mixer: its {m.kv_heads} value heads of {m.vdim} cannot be mixed "
                                   f"with the first such layer's {first.kv_heads} of {first.vdim}")
             l = BeralixLayer(replace(m, mix_role="first" if m is first else "later"), l.mlp)

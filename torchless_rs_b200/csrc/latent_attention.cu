@@ -778,7 +778,7 @@ extern "C" int tl_latent_attn_mma(const float* qa, int ld_qa, int qa_head, const
 }
 
 // ---------------------------------------------------------------------------
-// The per-head products on tensor cores (bfloat16 build), for steps of many tokens:
+// The per-head products on tensor cores (bfloat16 build):
 //   C[t, h, n] = gate * sum_k A[t, h, k] W[h, n, k],  A 32-bit (rounded to bfloat16 on its way into shared
 // memory), W bfloat16; C bfloat16, with the output gate of the kernels above if there is one (the value
 // up-projection), or 32-bit without a gate (OUT32: queries on their way into the latent space).  A block computes 64 rows x 64 outputs of
@@ -873,6 +873,75 @@ headwise_mma_kernel(const float* __restrict__ A, int lda, int a_head, const __nv
   }
 }
 
+// The same for few rows (M <= 16): a warp computes all rows of 8 outputs of one head, straight from memory to the
+// tensor cores' registers.  The order of the summation index is free as long as both operands take it alike, so a
+// lane reads eight neighbouring numbers of a weight row (16 bytes) and of its two rows of A and gives them to two
+// instructions.  KS warps share the summation (1 or 4; their sums meet in shared memory).  The first four pieces
+// of the weights, which no kernel of a step writes, are asked for before the wait for the kernels ahead.
+template <bool OUT32, int KS>
+__global__ void __launch_bounds__(128)
+headwise_few_kernel(const float* __restrict__ A, int lda, int a_head, const __nv_bfloat16* __restrict__ W,
+                    void* __restrict__ C, int ldc, int c_head, const float* __restrict__ G, int ldg, int g_one,
+                    int M, int N, int K) {
+  __shared__ float4 red[KS > 1 ? 4 : 1][32];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, qd = lane & 3;
+  const int h = blockIdx.z, n0 = (blockIdx.x * (4 / KS) + warp / KS) * 8, ks = warp % KS;
+  const __nv_bfloat16* wr = W + ((size_t)h * N + n0 + g) * K + qd * 8;
+  const bool live = n0 + g < N;
+  const int blocks = (K + 31) / 32;           // steps of 32 summands; this warp takes every KS-th from ks on
+  auto weights = [&](int kb) -> uint4 {
+    return live && kb * 32 + qd * 8 < K ? *reinterpret_cast<const uint4*>(wr + kb * 32) : make_uint4(0u, 0u, 0u, 0u);
+  };
+  uint4 w[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) w[i] = weights(ks + i * KS);
+  pdl_wait();
+  pdl_launch_dependents();
+  const float* Ar = A + (size_t)h * a_head + qd * 8;
+  const bool r0 = g < M, r1 = g + 8 < M;
+  float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+  for (int kb0 = ks; kb0 < blocks; kb0 += 4 * KS) {
+    if (kb0 != ks) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) w[i] = weights(kb0 + i * KS);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int k = (kb0 + i * KS) * 32;
+      const bool in = k + qd * 8 < K;
+      const float4 z4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      const float4* p0 = reinterpret_cast<const float4*>(Ar + (size_t)g * lda + k);
+      const float4* p1 = reinterpret_cast<const float4*>(Ar + (size_t)(g + 8) * lda + k);
+      const float4 x0 = in && r0 ? p0[0] : z4, x1 = in && r0 ? p0[1] : z4;
+      const float4 y0 = in && r1 ? p1[0] : z4, y1 = in && r1 ? p1[1] : z4;
+      const uint32_t a0[4] = {pack_bf16(x0.x, x0.y), pack_bf16(y0.x, y0.y), pack_bf16(x0.z, x0.w), pack_bf16(y0.z, y0.w)};
+      const uint32_t a1[4] = {pack_bf16(x1.x, x1.y), pack_bf16(y1.x, y1.y), pack_bf16(x1.z, x1.w), pack_bf16(y1.z, y1.w)};
+      mma_bf16(acc, a0, w[i].x, w[i].y);
+      mma_bf16(acc, a1, w[i].z, w[i].w);
+    }
+  }
+  if (KS > 1) {
+    red[KS > 1 ? warp : 0][lane] = make_float4(acc[0], acc[1], acc[2], acc[3]);
+    __syncthreads();
+    if (ks != 0) return;
+#pragma unroll
+    for (int i = 1; i < KS; ++i) {
+      const float4 v = red[KS > 1 ? warp + i : 0][lane];
+      acc[0] += v.x; acc[1] += v.y; acc[2] += v.z; acc[3] += v.w;
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const int m = g + 8 * (e >> 1), n = n0 + qd * 2 + (e & 1);
+    if (m >= M || n >= N) continue;
+    const size_t at = (size_t)m * ldc + (size_t)h * c_head + n;
+    if (OUT32) ((float*)C)[at] = acc[e];
+    else
+      ((__nv_bfloat16*)C)[at] =
+          __float2bfloat16_rn(G != nullptr ? acc[e] * hw_gate(G, ldg, g_one, m, h, n, N) : acc[e]);
+  }
+}
+
 // Returns TL_ERR_UNSUPPORTED for sizes or alignments it does not take (the FFMA kernel then runs).
 extern "C" int tl_headwise_mma(const float* A, int lda, int a_head, const void* W, void* C, int ldc, int c_head,
                                const float* G, int ldg, int g_one, int M, int N, int K, int heads, int out32,
@@ -882,6 +951,15 @@ extern "C" int tl_headwise_mma(const float* A, int lda, int a_head, const void* 
       ((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((uintptr_t)C & (out32 ? 7 : 3)) || heads > 65535 ||
       (M + HM_BM - 1) / HM_BM > 65535)
     return TL_ERR_UNSUPPORTED;
+  if (M <= 16) {
+#define FEW(OUT32_, KS_)                                                                                            \
+    return tl_launch(headwise_few_kernel<OUT32_, KS_>, dim3(((N + 7) / 8 * KS_ + 3) / 4, 1, heads), dim3(128), 0, \
+                     stream, A, lda, a_head, (const __nv_bfloat16*)W, C, ldc, c_head, G, ldg, g_one, M, N, K)
+    if (K >= 256) { if (out32) FEW(true, 4); FEW(false, 4); }
+    if (out32) FEW(true, 1);
+    FEW(false, 1);
+#undef FEW
+  }
   dim3 grid((N + HM_BN - 1) / HM_BN, (M + HM_BM - 1) / HM_BM, heads);
   return tl_launch(out32 ? headwise_mma_kernel<true> : headwise_mma_kernel<false>, grid, dim3(128), 0, stream, A, lda,
                    a_head, (const __nv_bfloat16*)W, C, ldc, c_head, G, ldg, g_one, M, N, K);

@@ -57,39 +57,57 @@ __device__ __forceinline__ void ln_stats(const float (&v)[K][4], int H, float ep
 }
 
 // ADD: y is normed with (w, b) and added to x in place; with w2 the new x is normed with (w2, b2) into `out`.
-// Otherwise row rows[r] (or r) of x is normed with (w, b) into row r of `out`.
-template <int K, bool ADD>
-__global__ void __launch_bounds__(1024)
+// Otherwise row rows[r] (or r) of x is normed with (w, b) into row r of `out`.  A block takes every gridDim.x-th
+// row, so that weights and biases are fetched once for all of them, and asks for its next row while it works on
+// one.
+template <int K, bool ADD, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 layernorm_vec_kernel(const float* __restrict__ y, int ldy, float* __restrict__ x, const int* __restrict__ rows,
                      const float* __restrict__ w, const float* __restrict__ b, float eps,
                      const float* __restrict__ w2, const float* __restrict__ b2, float eps2,
-                     act_t* __restrict__ out, int H) {
+                     act_t* __restrict__ out, int n_rows, int H) {
+  constexpr int KA = ADD ? K : 1;
   __shared__ float scratch[64];
-  float wv[K][4], bv[K][4];
-#pragma unroll
-  for (int j = 0; j < K; ++j) {
-    const int i = 4 * (threadIdx.x + j * blockDim.x);
-    if (i < H) { ln_load4(w + i, wv[j]); ln_load4(b + i, bv[j]); }
-  }
-  pdl_wait();
-  pdl_launch_dependents();
-  const size_t r = blockIdx.x;
-  float* xr = x + (size_t)(!ADD && rows != nullptr ? rows[r] : r) * H;
-  const float* src = ADD ? y + r * ldy : xr;
-  float v[K][4], xs[ADD ? K : 1][4];
+  float wv[K][4], bv[K][4], wv2[KA][4], bv2[KA][4];
+  const bool next = ADD && w2 != nullptr;
 #pragma unroll
   for (int j = 0; j < K; ++j) {
     const int i = 4 * (threadIdx.x + j * blockDim.x);
     if (i < H) {
-      ln_load4(src + i, v[j]);
-      if (ADD) ln_load4(xr + i, xs[ADD ? j : 0]);
-    } else {
-      v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.0f;
+      ln_load4(w + i, wv[j]);
+      ln_load4(b + i, bv[j]);
+      if (next) { ln_load4(w2 + i, wv2[ADD ? j : 0]); ln_load4(b2 + i, bv2[ADD ? j : 0]); }
     }
   }
-  float mean, inv;
-  ln_stats<K>(v, H, eps, scratch, 0, &mean, &inv);
-  if (!ADD) {
+  pdl_wait();
+  pdl_launch_dependents();
+  float v[K][4], xs[KA][4], nv[K][4], nx[KA][4];
+  auto fetch = [&](int r) {
+    const float* xr = x + (size_t)(!ADD && rows != nullptr ? rows[r] : r) * H;
+    const float* src = ADD ? y + (size_t)r * ldy : xr;
+#pragma unroll
+    for (int j = 0; j < K; ++j) {
+      const int i = 4 * (threadIdx.x + j * blockDim.x);
+      if (i < H) {
+        ln_load4(src + i, nv[j]);
+        if (ADD) ln_load4(xr + i, nx[ADD ? j : 0]);
+      } else {
+        nv[j][0] = nv[j][1] = nv[j][2] = nv[j][3] = 0.0f;
+      }
+    }
+  };
+  fetch(blockIdx.x);
+  for (int r = blockIdx.x; r < n_rows; r += gridDim.x) {
+#pragma unroll
+    for (int j = 0; j < K; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        v[j][e] = nv[j][e];
+        if (ADD) xs[ADD ? j : 0][e] = nx[ADD ? j : 0][e];
+      }
+    if (r + (int)gridDim.x < n_rows) fetch(r + gridDim.x);
+    float mean, inv;
+    ln_stats<K>(v, H, eps, scratch, 0, &mean, &inv);
 #pragma unroll
     for (int j = 0; j < K; ++j) {
       const int i = 4 * (threadIdx.x + j * blockDim.x);
@@ -97,31 +115,27 @@ layernorm_vec_kernel(const float* __restrict__ y, int ldy, float* __restrict__ x
         float o[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[e] = fmaf((v[j][e] - mean) * inv, wv[j][e], bv[j][e]);
-        ln_store4(out + r * H + i, o);
+        if (ADD) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[j][e] = xs[ADD ? j : 0][e] + o[e];
+          ln_store4(x + (size_t)r * H + i, v[j]);
+        } else {
+          ln_store4(out + (size_t)r * H + i, o);
+        }
       }
     }
-    return;
-  }
+    if (!next) continue;
+    ln_stats<K>(v, H, eps2, scratch, 2, &mean, &inv);
 #pragma unroll
-  for (int j = 0; j < K; ++j) {
-    const int i = 4 * (threadIdx.x + j * blockDim.x);
-    if (i < H) {
+    for (int j = 0; j < K; ++j) {
+      const int i = 4 * (threadIdx.x + j * blockDim.x);
+      if (i < H) {
+        float o[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[j][e] = xs[ADD ? j : 0][e] + fmaf((v[j][e] - mean) * inv, wv[j][e], bv[j][e]);
-      ln_store4(xr + i, v[j]);
-      if (w2 != nullptr) { ln_load4(w2 + i, wv[j]); ln_load4(b2 + i, bv[j]); }
-    }
-  }
-  if (w2 == nullptr) return;
-  ln_stats<K>(v, H, eps2, scratch, 2, &mean, &inv);
-#pragma unroll
-  for (int j = 0; j < K; ++j) {
-    const int i = 4 * (threadIdx.x + j * blockDim.x);
-    if (i < H) {
-      float o[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[e] = fmaf((v[j][e] - mean) * inv, wv[j][e], bv[j][e]);
-      ln_store4(out + r * H + i, o);
+        for (int e = 0; e < 4; ++e)
+          o[e] = fmaf((v[j][e] - mean) * inv, wv2[ADD ? j : 0][e], bv2[ADD ? j : 0][e]);
+        ln_store4(out + (size_t)r * H + i, o);
+      }
     }
   }
 }
@@ -168,16 +182,17 @@ static int ln_launch(const float* y, int ldy, float* x, const int* rows, const f
                      cudaStream_t stream) {
   const uintptr_t at = (uintptr_t)y | (uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)w2 | (uintptr_t)b2 |
                        (uintptr_t)out;
-  if (H % 4 == 0 && ldy % 4 == 0 && H <= 16384 && (at & 15) == 0) {
-#define LN_VEC(K_, THREADS_)                                                                                     \
-    return tl_launch(layernorm_vec_kernel<K_, ADD>, dim3(n_rows), dim3(THREADS_), 0, stream, y, ldy, x, rows, w, \
-                     b, eps, w2, b2, eps2, out, H)
+  if (H % 4 == 0 && ldy % 4 == 0 && H <= 8192 && (at & 15) == 0) {
+    // few rows: as many threads a row as it has pieces; many: fewer, so that several rows are in flight on an SM
+    const int grid = n_rows < 148 * 4 ? n_rows : 148 * 4;
+#define LN_VEC(K_, THREADS_)                                                                                      \
+    return tl_launch(layernorm_vec_kernel<K_, ADD, THREADS_>, dim3(grid), dim3(THREADS_), 0, stream, y, ldy, x, rows, w, b, \
+                     eps, w2, b2, eps2, out, n_rows, H)
     if (H <= 512) LN_VEC(1, 128);
     if (H <= 1024) LN_VEC(1, 256);
-    if (H <= 2048) LN_VEC(1, 512);
-    if (H <= 4096) LN_VEC(2, 512);
-    if (H <= 8192) LN_VEC(2, 1024);
-    LN_VEC(4, 1024);
+    if (H <= 2048) { if (n_rows < 148) LN_VEC(1, 512); LN_VEC(2, 256); }
+    if (H <= 4096) { if (n_rows < 148) LN_VEC(1, 1024); LN_VEC(2, 512); }
+    LN_VEC(2, 1024);
 #undef LN_VEC
   }
   return tl_launch(layernorm_any_kernel<ADD>, dim3(n_rows), dim3(H >= 2048 ? 512 : 128), 0, stream, y, ldy, x, rows, w,

@@ -425,8 +425,8 @@ class CoreOps:
             if gate.shape not in ((M, heads * N), (M, heads)) or gate.stride(1) != 1:
                 raise KernelError("headwise_gemm: the gate must be [rows, heads * outputs] or [rows, heads]")
             ldg, per_head = gate.stride(0), int(gate.shape[1] == heads)
-        if M > 16 and self.act_dtype == torch.bfloat16:
-            # many rows: the tensor-core kernel, where sizes and alignments allow it
+        if self.act_dtype == torch.bfloat16:
+            # the tensor-core kernels, where sizes and alignments allow them
             self.lib.tl_headwise_mma.restype = c_int
             st = self.lib.tl_headwise_mma(_ptr(a), c_int(a.stride(0)), c_int(a_head), _ptr(w), _ptr(c),
                                           c_int(c.stride(0)), c_int(c_head), _ptr(gate), c_int(ldg),
@@ -1259,7 +1259,7 @@ class CoreOps:
         _check(self._tl_selective_scan(
             _ptr(x), c_int(x.stride(0)), _ptr(zdt), _ptr(dt_bias), _ptr(bc), c_int(bc.stride(0)), c_int(col_b), _ptr(neg_a),
             _ptr(D), _ptr(z), c_int(z.stride(0)), _ptr(state), _ptr(y), _ptr(seq_start), _ptr(seq_slot),
-            c_int(seq_slot.numel()), c_int(channels), c_int(N), _stream()), "selective_scan")
+            c_int(T), c_int(seq_slot.numel()), c_int(channels), c_int(N), _stream()), "selective_scan")
 
 
 class SamplingOps:

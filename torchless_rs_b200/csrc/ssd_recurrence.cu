@@ -156,10 +156,123 @@ extern "C" int TL_NAME(tl_ssd_prep)(const float* z, int ld, int col_x, int col_d
                                 seq_slot, T, B, channels, H, stream);
 }
 
+// The convolution alone, four channels per thread (16- or 8-byte loads, kept as they came until they are used)
+// over a strip of SSD_STRIP tokens.  Everything else as in ssd_prep_kernel.
+#if TL_DTYPE == 0
+typedef float4 ssd_quad;
+__device__ __forceinline__ float ssd_fast_silu(float z) { return ssd_silu(z); }
+#else
+typedef uint2 ssd_quad;
+__device__ __forceinline__ float ssd_fast_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+#endif
+__device__ __forceinline__ void ssd_unpack(const float4& f, float (&v)[4]) {
+  v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+}
+__device__ __forceinline__ void ssd_unpack(const uint2& u, float (&v)[4]) {
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+__device__ __forceinline__ void ssd_store4(float* p, const float (&v)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void ssd_store4(__nv_bfloat16* p, const float (&v)[4]) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  uint2 u;
+  u.x = *reinterpret_cast<const uint32_t*>(&a);
+  u.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+template <int TAPS>
+__global__ void __launch_bounds__(128)
+conv_silu_vec_kernel(const act_t* __restrict__ z, int ld, const float* __restrict__ taps_w,
+                     const float* __restrict__ bias, float* __restrict__ kept, act_t* __restrict__ out,
+                     const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int B, int channels) {
+  const int c = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+  float w[4 * TAPS], bi[4] = {0.0f, 0.0f, 0.0f, 0.0f};      // w: channel after channel, its taps in a row
+  if (c < channels) {                       // weights: asked for before the wait
+    ssd_unpack(*reinterpret_cast<const float4*>(bias + c), bi);
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) {
+      float q[4];
+      ssd_unpack(*reinterpret_cast<const float4*>(taps_w + (size_t)c * TAPS + 4 * i), q);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) w[4 * i + e] = q[e];
+    }
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  int b, t0, n, strip;
+  if (!ssd_find_piece(blockIdx.x, SSD_STRIP, seq_start, B, &b, &t0, &n, &strip) || c >= channels) return;
+  float* mine = kept + (size_t)seq_slot[b] * (TAPS - 1) * channels + c;
+  const int count = seq_start[b + 1] - seq_start[b];
+  // the strip's inputs, and the TAPS - 1 ahead of it: inputs of the step, or, for the first strip, kept ones
+  ssd_quad raw[SSD_STRIP + TAPS - 1];
+  const act_t* zc = z + (size_t)t0 * ld + c;
+#pragma unroll
+  for (int i = 0; i < SSD_STRIP + TAPS - 1; ++i)
+    if ((i >= TAPS - 1 || strip > 0) && i < n + TAPS - 1)
+      raw[i] = *reinterpret_cast<const ssd_quad*>(zc + (ptrdiff_t)(i - (TAPS - 1)) * ld);
+  float before[TAPS - 1][4];
+#pragma unroll
+  for (int i = 0; i < TAPS - 1; ++i) {
+    if (strip > 0) ssd_unpack(raw[i], before[i]);
+    else ssd_unpack(*reinterpret_cast<const float4*>(mine + (size_t)i * channels), before[i]);
+  }
+  if (strip == 0) {
+    // this thread alone looks at the kept inputs, so it can replace them: the last TAPS - 1 of [kept | step]
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) {
+      const int j = count - (TAPS - 1) + i;          // place in the step; negative: kept from before
+      float v[4];
+      if (j >= 0) ssd_unpack(*reinterpret_cast<const ssd_quad*>(zc + (size_t)j * ld), v);
+      else {
+#pragma unroll
+        for (int q = 0; q < TAPS - 1; ++q)
+          if (q == TAPS - 1 + j) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] = before[q][e];
+          }
+      }
+      ssd_store4(mine + (size_t)i * channels, v);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < SSD_STRIP; ++j) {
+    if (j >= n) break;
+    float cur[4], o[4];
+    ssd_unpack(raw[j + TAPS - 1], cur);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float acc = bi[e];
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i) acc = fmaf(w[e * TAPS + i], before[i][e], acc);
+      o[e] = ssd_fast_silu(fmaf(w[e * TAPS + TAPS - 1], cur[e], acc));
+    }
+    ssd_store4(out + (size_t)(t0 + j) * channels + c, o);
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) before[i][e] = i + 1 < TAPS - 1 ? before[i + 1 < TAPS - 1 ? i + 1 : 0][e] : cur[e];
+  }
+}
+
 // The convolution alone: out [T, channels] = silu(conv(z[:, col_x:]) + bias), z in the activation type.
 extern "C" int TL_NAME(tl_conv_silu)(const void* z, int ld, int col_x, const float* taps_w, const float* bias, int taps,
                                      float* kept, void* out, const int* seq_start, const int* seq_slot, int T, int B,
                                      int channels, cudaStream_t stream) {
+  if (T <= 0 || B <= 0) return 0;
+  const uintptr_t at = (uintptr_t)z | (uintptr_t)kept | (uintptr_t)out | (uintptr_t)bias | (uintptr_t)taps_w;
+  if (taps >= 2 && taps <= 4 && channels > 0 && channels % 4 == 0 && ld % 4 == 0 && col_x % 4 == 0 && (at & 15) == 0) {
+    const dim3 grid(T / SSD_STRIP + B, (channels / 4 + 127) / 128);
+#define CONV(TAPS_)                                                                                                  \
+    return tl_launch(conv_silu_vec_kernel<TAPS_>, grid, dim3(128), 0, stream, (const act_t*)z + col_x, ld, taps_w,  \
+                     bias, kept, (act_t*)out, seq_start, seq_slot, B, channels)
+    if (taps == 2) CONV(2);
+    if (taps == 3) CONV(3);
+    CONV(4);
+#undef CONV
+  }
   return ssd_prep_launch<act_t>((const act_t*)z, ld, col_x, 0, taps_w, bias, taps, kept, out, nullptr, nullptr, nullptr,
                                 seq_start, seq_slot, T, B, channels, 0, stream);
 }
